@@ -5,7 +5,7 @@
 #include <cstdlib>
 #include <vector>
 extern "C" {
-void* xrh_cache_create(int, const int*, int, int, int, int, int32_t**);
+void* xrh_cache_create(int, const int*, const int*, int, int, int, int, int32_t**);
 void xrh_cache_destroy(void*);
 int xrh_open(void*); int xrh_close(void*, int); long long xrh_length(void*, int);
 int xrh_can_reserve(void*, int, long long); int xrh_reserve(void*, int, long long); int xrh_commit(void*, int); int xrh_cancel(void*, int);
@@ -16,10 +16,10 @@ int main() {
     srand(1);
     for (int trial = 0; trial < 200; trial++) {
         int G = 1 + rand() % 2, ps = 1 << (rand() % 5), n_pages = 8 + rand() % 30, mr = 1 + rand() % 5, mp = 12;
-        int windows[2] = {-1, 3 + rand() % 20};
+        int windows[2] = {-1, 3 + rand() % 20}, keeps[2] = {0, rand() % 3 ? rand() % 12 : 0};
         std::vector<std::vector<int32_t>> tabs(G, std::vector<int32_t>((size_t)mr * mp));
         int32_t* tp[2] = {tabs[0].data(), G > 1 ? tabs[1].data() : nullptr};
-        void* c = xrh_cache_create(G, windows, n_pages, ps, mr, mp, tp);
+        void* c = xrh_cache_create(G, windows, keeps, n_pages, ps, mr, mp, tp);
         std::vector<int> open;
         char msg[256];
         for (int it = 0; it < 2000; it++) {

@@ -8,7 +8,9 @@ all keys (``window is None``) or the last ``window`` keys (the reference's
 per-layer sliding flag, src/model.h:229-235).  Every group has a pool of its
 own and every request a block table per group.  Pages go back to the pool
 when a request ends, and -- in a window group -- as soon as every position in
-the page lies behind the window of every query still to come.
+the page lies behind the window of every query still to come.  A window group
+may keep a request's first positions visible from anywhere (``keep_first``);
+the pages that hold those stay until the request ends.
 
 The bookkeeping itself is native code (``csrc/host/page_cache.cpp``, built into
 ``libxrhost.so`` and called through ctypes); this module gives it its Python
@@ -41,7 +43,7 @@ def host_lib() -> ctypes.CDLL:
         sig = {
             "xrh_pool_create": (vp, [i]), "xrh_pool_destroy": (None, [vp]), "xrh_pool_n_free": (i, [vp]),
             "xrh_pool_take": (i, [vp]), "xrh_pool_give": (i, [vp, i]),
-            "xrh_cache_create": (vp, [i, vp, i, i, i, i, vp]), "xrh_cache_destroy": (None, [vp]),
+            "xrh_cache_create": (vp, [i, vp, vp, i, i, i, i, vp]), "xrh_cache_destroy": (None, [vp]),
             "xrh_has_free_slot": (i, [vp]), "xrh_n_free": (i, [vp, i]), "xrh_high_water": (i, [vp, i]),
             "xrh_pool_take_of": (i, [vp, i]), "xrh_pool_give_of": (i, [vp, i, i]),
             "xrh_open": (i, [vp]), "xrh_close": (i, [vp, i]), "xrh_length": (ll, [vp, i]), "xrh_reserved": (ll, [vp, i]),
@@ -67,9 +69,11 @@ class CacheError(RuntimeError):
 
 @dataclass(frozen=True)
 class GroupSpec:
-    """Layers with the same need.  `window` None keeps every key."""
+    """Layers with the same need.  `window` None keeps every key; with a window, the first `keep_first` positions of a request
+    are kept all the same."""
     name: str
     window: Optional[int] = None
+    keep_first: int = 0
 
 
 class PagePool:
@@ -149,8 +153,9 @@ class CacheManager:
         G = len(self.groups)
         self._L = host_lib()
         windows = (ctypes.c_int * max(G, 1))(*[-1 if g.window is None else int(g.window) for g in self.groups])
+        keeps = (ctypes.c_int * max(G, 1))(*[0 if g.window is None else int(g.keep_first) for g in self.groups])
         self._table_ptrs = (ctypes.c_void_p * max(G, 1))(*[t.ctypes.data for t in self.tables])
-        self._h = self._L.xrh_cache_create(G, windows, n_pages, page_size, max_requests, self.max_pages_per_request,
+        self._h = self._L.xrh_cache_create(G, windows, keeps, n_pages, page_size, max_requests, self.max_pages_per_request,
                                            self._table_ptrs)
         if not self._h:
             raise CacheError("the cache manager could not be made (sizes must be positive)")

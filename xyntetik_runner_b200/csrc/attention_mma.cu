@@ -2,7 +2,8 @@
 // accumulation), for prompt portions and for decoded tokens, head sizes 16..128 in steps of 16.
 //
 // For the query at position p, head h, kv head h / (H/K):  s_t = (q . k_t) * scale over the keys
-// t0 <= t <= p (t0 = max(0, p - window + 1), or 0), a = softmax(s), o = sum_t a_t v_t
+// t0 <= t <= p (t0 = max(0, p - window + 1), or 0), a = softmax(s), o = sum_t a_t v_t, with kept first keys and a bias by
+// distance as options (attention_mask.cuh)
 // (src/model.c:3548-3589, 3409-3415).  The reference's kernels are `k_attn` (one block per head and
 // token, scores through a global scratch, src/kernels.cu:2043-2141) and the split `k_attn_dec` +
 // `k_attn_merge` for decoding (src/kernels.cu:2171-2270).
@@ -26,6 +27,7 @@
 // (k_attention_keys_tma: spans, combined inside a cluster where all of them are resident at once;
 // k_attention_keys_even: the tiles of all requests cut into one equal run per resident CTA, for many or unequal requests).
 #include "common.cuh"
+#include "attention_mask.cuh"
 #include <math.h>
 #include <cuda.h>
 
@@ -57,6 +59,8 @@ struct AttnMmaArgs {
     int recv_rows;               // cluster variant: most packed rows any request of the step has (sizes what a block receives)
     const float* sink;           // [H] or null: a logit per query head that joins the softmax's denominator once (no key, no value)
     float softcap;               // c > 0: every score becomes c tanh(score / c); 0: scores as they are
+    int keep_first;              // with a window: the first keys that stay visible behind it (their tiles belong to a request's first span)
+    XrBias bias;
 };
 
 // c tanh(x / c) through one exponential: tanh(y) = 1 - 2 / (exp(2y) + 1), exact in the limits and within a few 1e-7 elsewhere.
@@ -132,7 +136,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 
 // Gather one tile of keys AND values [ATT_TILE][HD] each into shared memory rows of HD + 8 elements.
-// Rows at positions outside [lo, hi] or on a page the request no longer holds are zero-filled.
+// Rows at positions outside [lo, hi] (but for the kept first keys) or on a page the request no longer holds are zero-filled.
 // A thread keeps one 16-byte column and walks rows, so the page of a row is looked up once for K and V.
 template <int HD>
 __device__ __forceinline__ void load_kv_tile(__nv_bfloat16* kdst, __nv_bfloat16* vdst, const AttnMmaArgs& a, const int* bt,
@@ -147,7 +151,7 @@ __device__ __forceinline__ void load_kv_tile(__nv_bfloat16* kdst, __nv_bfloat16*
     for (int r = r0; r < ATT_TILE; r += RPP) {
         int kp = key0 + r;
         int page = -1, off = 0;
-        if (kp >= lo && kp <= hi) {
+        if (xr_sees(kp, hi, lo, a.keep_first)) {
             int pi;
             if (a.page_shift >= 0) { pi = kp >> a.page_shift; off = kp & (a.page_size - 1); }
             else { pi = kp / a.page_size; off = kp - pi * a.page_size; }
@@ -196,14 +200,33 @@ __device__ __forceinline__ const __nv_bfloat16* tile_ptr(const __nv_bfloat16* ba
     return base + row * (HD + 8) + col;
 }
 
+//
+// s comes in as what the scores start from: the bias by distance (tile_start), or zero.
+// bias_a, bias_b: the rows of the bias table of this lane's two query rows (null: no bias)
+template <int NKT, bool LOWER_ONLY = false>
+__device__ __forceinline__ void tile_start(float (*s)[4], const float* bias_a, const float* bias_b, int bias_len, int key_first, int pos_a, int pos_b) {
+    if (bias_a == nullptr) {
+#pragma unroll
+        for (int j = 0; j < NKT; j++) { s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f; }
+        return;
+    }
+    const int t2 = (threadIdx.x & 3) * 2;
+#pragma unroll
+    for (int j = 0; j < NKT; j++) {
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            const int kp = key_first + j * 8 + t2 + e;
+            s[j][e] = xr_bias_at(bias_a, bias_len, pos_a - kp);
+            s[j][2 + e] = LOWER_ONLY ? 0.f : xr_bias_at(bias_b, bias_len, pos_b - kp);
+        }
+    }
+}
+
 template <int HD, int NKT, bool LOWER_ONLY = false, bool SWZ = false>
 __device__ __forceinline__ void tile_step(const uint32_t (*qf)[4], const __nv_bfloat16* ks, const __nv_bfloat16* vs,
-                                          int col0, int key0, int pos_a, int pos_b, int window, float scale, float cap,
-                                          float* m, float* l, float (*o)[4]) {
+                                          int col0, int key0, int pos_a, int pos_b, int window, int keep_first, float scale, float cap,
+                                          float* m, float* l, float (*o)[4], float (*s)[4]) {
     const int lane = threadIdx.x & 31;
-    float s[NKT][4];
-#pragma unroll
-    for (int j = 0; j < NKT; j++) { s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f; }
 #pragma unroll
     for (int kk = 0; kk < HD / 16; kk++) {
 #pragma unroll
@@ -234,11 +257,11 @@ __device__ __forceinline__ void tile_step(const uint32_t (*qf)[4], const __nv_bf
 #pragma unroll
         for (int e = 0; e < 2; e++) {
             int kp = key0 + col0 + j * 8 + t2 + e;
-            float va = (kp <= pos_a && kp >= lo_a) ? s[j][e] * scale : -INFINITY;
+            float va = xr_sees(kp, pos_a, lo_a, keep_first) ? s[j][e] * scale : -INFINITY;
             s[j][e] = va;
             mx_a = fmaxf(mx_a, va);
             if (!LOWER_ONLY) {
-                float vb = (kp <= pos_b && kp >= lo_b) ? s[j][2 + e] * scale : -INFINITY;
+                float vb = xr_sees(kp, pos_b, lo_b, keep_first) ? s[j][2 + e] * scale : -INFINITY;
                 s[j][2 + e] = vb;
                 mx_b = fmaxf(mx_b, vb);
             }
@@ -296,6 +319,11 @@ __device__ __forceinline__ void tile_step(const uint32_t (*qf)[4], const __nv_bf
     }
 }
 
+// The bias table's row of packed row pr's query head (null: no bias).
+__device__ __forceinline__ const float* att_bias_row(const AttnMmaArgs& a, int kvh, int pr) {
+    return a.bias.table != nullptr ? a.bias.table + (size_t)(kvh * a.G + pr % a.G) * a.bias.len : nullptr;
+}
+
 // Q rows of this CTA -> shared [ATT_ROWS or 16][HD + 8]; rows past the portion are zero.
 template <int HD>
 __device__ __forceinline__ void load_q(__nv_bfloat16* qs, const AttnMmaArgs& a, int tok_base, int kvh, int row0, int rows,
@@ -349,8 +377,9 @@ k_attention_rows(AttnMmaArgs a, int n_seg) {
     const int last_row = min(rows_total, row0 + ATT_ROWS) - 1;
     const int hi = pos0 + last_row / a.G;                                            // last key any row may read
     const int lo = a.window > 0 ? max(0, pos0 + row0 / a.G - a.window + 1) : 0;       // first key any row may read
-    const int t_lo = lo / ATT_TILE, t_hi = hi / ATT_TILE;
-    load_kv_tile<HD>(kbuf, vbuf, a, bt, kvh, t_lo * ATT_TILE, lo, hi);
+    const int t_lo = lo / ATT_TILE, t_hi = hi / ATT_TILE, kept_tiles = xr_kept_tiles(a.keep_first, lo, ATT_TILE);
+    const int n_tiles = kept_tiles + t_hi - t_lo + 1;
+    load_kv_tile<HD>(kbuf, vbuf, a, bt, kvh, xr_walk_tile(0, kept_tiles, t_lo) * ATT_TILE, lo, hi);
     cp_async_commit();
     __syncthreads();
     uint32_t qf[HD / 16][4];
@@ -365,20 +394,26 @@ k_attention_rows(AttnMmaArgs a, int n_seg) {
     for (int d = 0; d < HD / 8; d++) { o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f; }
     // a warp whose rows all end before a tile starts has nothing to do in it
     const int warp_hi = pos0 + min(last_row, row0 + warp * 16 + 15) / a.G;
+    const float* bias_a = att_bias_row(a, kvh, ra);
+    const float* bias_b = att_bias_row(a, kvh, rb);
 
-    for (int t = t_lo; t <= t_hi; t++) {
-        int cur = (t - t_lo) & 1;
-        if (t < t_hi) {
-            load_kv_tile<HD>(kbuf + (cur ^ 1) * ATT_TILE * LD, vbuf + (cur ^ 1) * ATT_TILE * LD, a, bt, kvh, (t + 1) * ATT_TILE, lo, hi);
+    for (int i = 0; i < n_tiles; i++) {
+        const int cur = i & 1, t = xr_walk_tile(i, kept_tiles, t_lo);
+        if (i + 1 < n_tiles) {
+            load_kv_tile<HD>(kbuf + (cur ^ 1) * ATT_TILE * LD, vbuf + (cur ^ 1) * ATT_TILE * LD, a, bt, kvh,
+                             xr_walk_tile(i + 1, kept_tiles, t_lo) * ATT_TILE, lo, hi);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
             cp_async_wait<0>();
         }
         __syncthreads();
-        if (t * ATT_TILE <= warp_hi)
+        if (t * ATT_TILE <= warp_hi) {
+            float s[8][4];
+            tile_start<8>(s, bias_a, bias_b, a.bias.len, t * ATT_TILE, pos_a, pos_b);
             tile_step<HD, 8>(qf, kbuf + cur * ATT_TILE * LD, vbuf + cur * ATT_TILE * LD, 0, t * ATT_TILE, pos_a, pos_b,
-                             a.window, a.scale, a.softcap, m, l, o);
+                             a.window, a.keep_first, a.scale, a.softcap, m, l, o, s);
+        }
         __syncthreads();
     }
     // rows a (lane/4) and b (+8): columns d*8 + 2*(lane%4) (+1)
@@ -425,12 +460,14 @@ k_attention_keys(AttnMmaArgs a) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
     load_q<HD>(qs, a, tok_base, kvh, 0, 16, rows_total);
-    const int t_lo = lo / ATT_TILE, t_hi = hi / ATT_TILE;
-    // ring of ATT_KSTAGES tiles: tiles t+1 .. t+ATT_KSTAGES-1 are in flight while tile t is used
+    // (the kept first keys' tiles belong to the first span)
+    const int t_lo = lo / ATT_TILE, t_hi = hi / ATT_TILE, kept_tiles = span == 0 ? xr_kept_tiles(a.keep_first, lo, ATT_TILE) : 0;
+    const int n_tiles = kept_tiles + t_hi - t_lo + 1;
+    // ring of ATT_KSTAGES tiles: the ATT_KSTAGES - 1 tiles behind the one in use are in flight
 #pragma unroll
     for (int i = 0; i < ATT_KSTAGES - 1; i++) {
-        if (t_lo + i <= t_hi)
-            load_kv_tile<HD>(kbuf + i * ATT_TILE * LD, vbuf + i * ATT_TILE * LD, a, bt, kvh, (t_lo + i) * ATT_TILE, lo, hi);
+        if (i < n_tiles)
+            load_kv_tile<HD>(kbuf + i * ATT_TILE * LD, vbuf + i * ATT_TILE * LD, a, bt, kvh, xr_walk_tile(i, kept_tiles, t_lo) * ATT_TILE, lo, hi);
         cp_async_commit();
     }
     __syncthreads();
@@ -445,24 +482,30 @@ k_attention_keys(AttnMmaArgs a) {
 #pragma unroll
     for (int d = 0; d < HD / 8; d++) { o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f; }
 
-    for (int t = t_lo; t <= t_hi; t++) {
-        int cur = (t - t_lo) % ATT_KSTAGES;
-        int nxt = (t - t_lo + ATT_KSTAGES - 1) % ATT_KSTAGES;
-        if (t + ATT_KSTAGES - 1 <= t_hi)
-            load_kv_tile<HD>(kbuf + nxt * ATT_TILE * LD, vbuf + nxt * ATT_TILE * LD, a, bt, kvh, (t + ATT_KSTAGES - 1) * ATT_TILE, lo, hi);
+    const float* bias_a = att_bias_row(a, kvh, ra);
+    const float* bias_b = att_bias_row(a, kvh, rb);
+    for (int i = 0; i < n_tiles; i++) {
+        const int t = xr_walk_tile(i, kept_tiles, t_lo);
+        int cur = i % ATT_KSTAGES;
+        int nxt = (i + ATT_KSTAGES - 1) % ATT_KSTAGES;
+        if (i + ATT_KSTAGES - 1 < n_tiles)
+            load_kv_tile<HD>(kbuf + nxt * ATT_TILE * LD, vbuf + nxt * ATT_TILE * LD, a, bt, kvh,
+                             xr_walk_tile(i + ATT_KSTAGES - 1, kept_tiles, t_lo) * ATT_TILE, lo, hi);
         cp_async_commit();
+        float s[2][4];
+        tile_start<2>(s, bias_a, bias_b, a.bias.len, t * ATT_TILE + warp * 16, pos_a, pos_b);
         cp_async_wait<ATT_KSTAGES - 1>();
         __syncthreads();
         // warp w takes keys [16w, 16w + 16) of the tile; every key of these tiles lies inside the span, and
         // keys outside [lo, hi] are outside every row's own range, so the per-row mask is all that is needed
         int c0 = warp * 16, kfirst = t * ATT_TILE + c0;
-        if (kfirst <= hi && kfirst + 15 >= lo) {
+        if (kfirst <= hi && (kfirst + 15 >= lo || kfirst < a.keep_first)) {
             if (rows_total <= 8)
                 tile_step<HD, 2, true>(qf, kbuf + cur * ATT_TILE * LD, vbuf + cur * ATT_TILE * LD, c0, t * ATT_TILE, pos_a, pos_b,
-                                       a.window, a.scale, a.softcap, m, l, o);
+                                       a.window, a.keep_first, a.scale, a.softcap, m, l, o, s);
             else
                 tile_step<HD, 2, false>(qf, kbuf + cur * ATT_TILE * LD, vbuf + cur * ATT_TILE * LD, c0, t * ATT_TILE, pos_a, pos_b,
-                                        a.window, a.scale, a.softcap, m, l, o);
+                                        a.window, a.keep_first, a.scale, a.softcap, m, l, o, s);
         }
         __syncthreads();
     }
@@ -573,7 +616,8 @@ k_attention_keys_tma(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs 
     const int lo = max(lo_all, k_begin), hi = min(hi_all, k_begin + SPAN - 1);
     const int* bt = a.block_tables + (size_t)seg * a.max_pages;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t_lo = lo / ATT_TILE, t_hi = hi / ATT_TILE;
+    const int t_lo = lo / ATT_TILE, t_hi = hi / ATT_TILE, kept_tiles = span == 0 ? xr_kept_tiles(a.keep_first, lo, ATT_TILE) : 0;
+    const int n_tiles = kept_tiles + t_hi - t_lo + 1;              // (the kept first keys' tiles belong to the first span)
     const int box_rows = a.page_size < ATT_TILE ? a.page_size : ATT_TILE;
 
     if (threadIdx.x == 0) {
@@ -609,10 +653,10 @@ k_attention_keys_tma(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs 
     // before the step's own tokens starts its copies before the kernel ahead in the stream is complete.
     const bool old_keys_only = hi < pos0;
     if (threadIdx.x == 0 && old_keys_only)
-        for (int i = 0; i < STAGES - 1 && t_lo + i <= t_hi; i++) fetch(t_lo + i, i);
+        for (int i = 0; i < STAGES - 1 && i < n_tiles; i++) fetch(xr_walk_tile(i, kept_tiles, t_lo), i);
     xr_pdl_wait();
     if (threadIdx.x == 0 && !old_keys_only)
-        for (int i = 0; i < STAGES - 1 && t_lo + i <= t_hi; i++) fetch(t_lo + i, i);
+        for (int i = 0; i < STAGES - 1 && i < n_tiles; i++) fetch(xr_walk_tile(i, kept_tiles, t_lo), i);
     load_q<HD>(qs, a, tok_base, kvh, 0, 16, rows_total);
     __syncthreads();
     uint32_t qf[HD / 16][4];
@@ -626,9 +670,13 @@ k_attention_keys_tma(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs 
 #pragma unroll
     for (int d = 0; d < HD / 8; d++) { o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f; }
 
-    for (int t = t_lo; t <= t_hi; t++) {
-        int i = t - t_lo, cur = i % STAGES;
-        if (threadIdx.x == 0 && t + STAGES - 1 <= t_hi) fetch(t + STAGES - 1, (i + STAGES - 1) % STAGES);
+    const float* bias_a = att_bias_row(a, kvh, ra);
+    const float* bias_b = att_bias_row(a, kvh, rb);
+    for (int i = 0; i < n_tiles; i++) {
+        const int t = xr_walk_tile(i, kept_tiles, t_lo), cur = i % STAGES;
+        if (threadIdx.x == 0 && i + STAGES - 1 < n_tiles) fetch(xr_walk_tile(i + STAGES - 1, kept_tiles, t_lo), (i + STAGES - 1) % STAGES);
+        float s[2][4];
+        tile_start<2>(s, bias_a, bias_b, a.bias.len, t * ATT_TILE + warp * 16, pos_a, pos_b);      // (on its way while the tile is)
         // A wait that runs out does not leave the loop (the threads of a CTA must keep meeting at the barriers
         // below); it is recorded, the result of this CTA is then meaningless, and the status word says so.
         if (!att_mbar_wait(&full[cur], (i / STAGES) & 1)) *gave_up = 1;
@@ -644,19 +692,20 @@ k_attention_keys_tma(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs 
             __syncthreads();
         }
         if (t * ATT_TILE < lo) {
-            int n_bad = lo - t * ATT_TILE;
-            for (int e = threadIdx.x; e < n_bad * (HD / 8); e += ATT_THREADS) {
+            // rows behind the kept keys and ahead of the window
+            const int bad0 = max(0, a.keep_first - t * ATT_TILE), bad1 = min(ATT_TILE, lo - t * ATT_TILE);
+            for (int e = bad0 * (HD / 8) + threadIdx.x; e < bad1 * (HD / 8); e += ATT_THREADS) {
                 int r = e / (HD / 8), c = (e % (HD / 8)) * 8;
                 *reinterpret_cast<uint4*>(const_cast<__nv_bfloat16*>(tile_ptr<HD, true>(vt, r, c))) = make_uint4(0, 0, 0, 0);
             }
             __syncthreads();
         }
         int c0 = warp * 16, kfirst = t * ATT_TILE + c0;
-        if (kfirst <= hi && kfirst + 15 >= lo) {
+        if (kfirst <= hi && (kfirst + 15 >= lo || kfirst < a.keep_first)) {
             if (rows_total <= 8)
-                tile_step<HD, 2, true, true>(qf, kbuf + cur * TILE_ELEMS, vt, c0, t * ATT_TILE, pos_a, pos_b, a.window, a.scale, a.softcap, m, l, o);
+                tile_step<HD, 2, true, true>(qf, kbuf + cur * TILE_ELEMS, vt, c0, t * ATT_TILE, pos_a, pos_b, a.window, a.keep_first, a.scale, a.softcap, m, l, o, s);
             else
-                tile_step<HD, 2, false, true>(qf, kbuf + cur * TILE_ELEMS, vt, c0, t * ATT_TILE, pos_a, pos_b, a.window, a.scale, a.softcap, m, l, o);
+                tile_step<HD, 2, false, true>(qf, kbuf + cur * TILE_ELEMS, vt, c0, t * ATT_TILE, pos_a, pos_b, a.window, a.keep_first, a.scale, a.softcap, m, l, o, s);
         }
         __syncthreads();                 // everyone is done with stage `cur` before it is fetched into again
     }
@@ -857,7 +906,7 @@ k_attention_keys_even(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs
         int cnt = 0;
         if (L > 0 && L * a.G <= 16) {
             const int lo = a.window > 0 ? max(0, p0 - a.window + 1) : 0;
-            cnt = (p0 + L - 1) / ATT_TILE - lo / ATT_TILE + 1;
+            cnt = xr_kept_tiles(a.keep_first, lo, ATT_TILE) + (p0 + L - 1) / ATT_TILE - lo / ATT_TILE + 1;
         }
         seg_pre[s + 1] = cnt;
     }
@@ -890,8 +939,14 @@ k_attention_keys_even(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs
     if (begin >= end) return;
     const int n_mine = (int)(end - begin);
 
-    // the pair and the tile at place f of the row of all tiles; t_first and cnt: the pair's first tile and its tiles
-    auto locate = [&](long long f, int& seg, int& kvh, int& t, int& t_first, int& cnt) {
+    // the pair at place f of the row of all tiles and the tile's place w in the pair's walk of cnt tiles: kept first tiles,
+    // then from t_lo on (xr_walk_tile)
+    auto walk_of = [&](int seg, int& kept_tiles, int& t_lo) {
+        const int p0 = a.seg_pos0[seg], lo = a.window > 0 ? max(0, p0 - a.window + 1) : 0;
+        t_lo = lo / ATT_TILE;
+        kept_tiles = xr_kept_tiles(a.keep_first, lo, ATT_TILE);
+    };
+    auto locate = [&](long long f, int& seg, int& kvh, int& w, int& kept_tiles, int& t_lo, int& cnt) {
         int lo = 0, hi = n_seg;                                    // K * seg_pre[lo] <= f < K * seg_pre[hi]
         while (hi - lo > 1) {
             const int mid = (lo + hi) >> 1;
@@ -901,17 +956,16 @@ k_attention_keys_even(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs
         cnt = seg_pre[lo + 1] - seg_pre[lo];
         const int rem = (int)(f - (long long)a.K * seg_pre[lo]);
         kvh = rem / cnt;
-        const int p0 = a.seg_pos0[lo];
-        t_first = (a.window > 0 ? max(0, p0 - a.window + 1) : 0) / ATT_TILE;
-        t = t_first + rem % cnt;
+        walk_of(lo, kept_tiles, t_lo);
+        w = rem % cnt;
     };
 
     // thread 0 keeps the place of the next tile to fetch; tile number i of the run goes to stage i % STAGES
     const int box_rows = a.page_size < ATT_TILE ? a.page_size : ATT_TILE;
-    int fs = 0, fk = 0, ft = 0, ft_first = 0, fcnt = 1, fetched = 0;
-    if (tid == 0) locate(begin, fs, fk, ft, ft_first, fcnt);
+    int fs = 0, fk = 0, fw = 0, fkept = 0, ft_lo = 0, fcnt = 1, fetched = 0;
+    if (tid == 0) locate(begin, fs, fk, fw, fkept, ft_lo, fcnt);
     auto fetch_next = [&]() {
-        const int s = fetched % STAGES;
+        const int s = fetched % STAGES, ft = xr_walk_tile(fw, fkept, ft_lo);
         const int* bt = a.block_tables + (size_t)fs * a.max_pages;
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      // the stage was read, and perhaps partly cleared, by threads
         asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(att_smem_u32(&full[s])), "r"(2 * TILE_ELEMS * 2) : "memory");
@@ -934,22 +988,21 @@ k_attention_keys_even(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs
             }
         }
         fetched++;
-        if (++ft == ft_first + fcnt) {                             // on to the next pair
+        if (++fw == fcnt) {                                        // on to the next pair
             if (++fk == a.K) {
                 fk = 0;
                 do { fs++; } while (fs < n_seg && seg_pre[fs + 1] == seg_pre[fs]);
                 if (fs < n_seg) {
-                    const int p0 = a.seg_pos0[fs];
                     fcnt = seg_pre[fs + 1] - seg_pre[fs];
-                    ft_first = (a.window > 0 ? max(0, p0 - a.window + 1) : 0) / ATT_TILE;
+                    walk_of(fs, fkept, ft_lo);
                 }
             }
-            ft = ft_first;
+            fw = 0;
         }
     };
     // tiles that hold keys of earlier steps only may be asked for before the kernel ahead in the stream is complete
     if (tid == 0)
-        while (fetched < STAGES && fetched < n_mine && (ft + 1) * ATT_TILE <= a.seg_pos0[fs]) fetch_next();
+        while (fetched < STAGES && fetched < n_mine && (xr_walk_tile(fw, fkept, ft_lo) + 1) * ATT_TILE <= a.seg_pos0[fs]) fetch_next();
     xr_pdl_wait();
     if (tid == 0)
         while (fetched < STAGES && fetched < n_mine) fetch_next();
@@ -957,14 +1010,13 @@ k_attention_keys_even(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs
     long long pos = begin;
     int i0 = 0;                                                    // number in the run of the piece's first tile
     while (pos < end) {
-        int seg, kvh, t_from, t_first, cnt;
-        locate(pos, seg, kvh, t_from, t_first, cnt);
+        int seg, kvh, w_from, kept_tiles, t_lo, cnt;
+        locate(pos, seg, kvh, w_from, kept_tiles, t_lo, cnt);
         const int L = a.seg_len[seg], rows_total = L * a.G, pos0 = a.seg_pos0[seg], tok_base = a.seg_start[seg];
         const int hi = pos0 + L - 1, lo = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
-        const int t_last = t_first + cnt - 1;
         const long long left = end - pos;
-        const int n_here = (long long)(t_last - t_from + 1) < left ? t_last - t_from + 1 : (int)left;
-        const int t_to = t_from + n_here - 1;
+        const int n_here = (long long)(cnt - w_from) < left ? cnt - w_from : (int)left;
+        const int w_to = w_from + n_here - 1;
         __syncthreads();                                           // the sums of the piece before have been read
         load_q<HD>(qs, a, tok_base, kvh, 0, 16, rows_total);
         __syncthreads();
@@ -979,8 +1031,12 @@ k_attention_keys_even(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs
 #pragma unroll
         for (int d = 0; d < HD / 8; d++) { o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f; }
 
-        for (int t = t_from; t <= t_to; t++) {
-            const int i = i0 + (t - t_from), cur = i % STAGES;
+        const float* bias_a = att_bias_row(a, kvh, ra);
+        const float* bias_b = att_bias_row(a, kvh, rb);
+        for (int w = w_from; w <= w_to; w++) {
+            const int t = xr_walk_tile(w, kept_tiles, t_lo), i = i0 + (w - w_from), cur = i % STAGES;
+            float s[2][4];
+            tile_start<2>(s, bias_a, bias_b, a.bias.len, t * ATT_TILE + warp * 16, pos_a, pos_b);  // (on its way while the tile is)
             if (!att_mbar_wait(&full[cur], (i / STAGES) & 1)) *gave_up = 1;
             __nv_bfloat16* vt = vbuf + cur * TILE_ELEMS;
             if ((t + 1) * ATT_TILE - 1 > hi) {
@@ -993,19 +1049,20 @@ k_attention_keys_even(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs
                 __syncthreads();
             }
             if (t * ATT_TILE < lo) {
-                const int n_bad = lo - t * ATT_TILE;
-                for (int e = tid; e < n_bad * (HD / 8); e += ATT_THREADS) {
+                // rows behind the kept keys and ahead of the window
+                const int bad0 = max(0, a.keep_first - t * ATT_TILE), bad1 = min(ATT_TILE, lo - t * ATT_TILE);
+                for (int e = bad0 * (HD / 8) + tid; e < bad1 * (HD / 8); e += ATT_THREADS) {
                     const int r = e / (HD / 8), cc = (e % (HD / 8)) * 8;
                     *reinterpret_cast<uint4*>(const_cast<__nv_bfloat16*>(tile_ptr<HD, true>(vt, r, cc))) = make_uint4(0, 0, 0, 0);
                 }
                 __syncthreads();
             }
             const int c0 = warp * 16, kfirst = t * ATT_TILE + c0;
-            if (kfirst <= hi && kfirst + 15 >= lo) {
+            if (kfirst <= hi && (kfirst + 15 >= lo || kfirst < a.keep_first)) {
                 if (rows_total <= 8)
-                    tile_step<HD, 2, true, true>(qf, kbuf + cur * TILE_ELEMS, vt, c0, t * ATT_TILE, pos_a, pos_b, a.window, a.scale, a.softcap, m, l, o);
+                    tile_step<HD, 2, true, true>(qf, kbuf + cur * TILE_ELEMS, vt, c0, t * ATT_TILE, pos_a, pos_b, a.window, a.keep_first, a.scale, a.softcap, m, l, o, s);
                 else
-                    tile_step<HD, 2, false, true>(qf, kbuf + cur * TILE_ELEMS, vt, c0, t * ATT_TILE, pos_a, pos_b, a.window, a.scale, a.softcap, m, l, o);
+                    tile_step<HD, 2, false, true>(qf, kbuf + cur * TILE_ELEMS, vt, c0, t * ATT_TILE, pos_a, pos_b, a.window, a.keep_first, a.scale, a.softcap, m, l, o, s);
             }
             __syncthreads();                                       // everyone is done with stage `cur`:
             if (tid == 0 && fetched < n_mine) fetch_next();        // tile i + STAGES goes into it at once, so the ring stays full
@@ -1043,7 +1100,7 @@ k_attention_keys_even(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs
                 }
             }
         }
-        if (t_from != t_first) {
+        if (w_from != 0) {
             // a later piece of a pair that began in a CTA before this one: leave it in this CTA's slot
             float* pacc = a.part_acc + (size_t)c * 16 * HD;
             float* pml = a.part_ml + (size_t)c * 32;
@@ -1059,7 +1116,7 @@ k_attention_keys_even(const __grid_constant__ CUtensorMap cache_map, AttnMmaArgs
             __syncthreads();
             if (tid == 0) { __threadfence(); att_st_release(flags + c, 1); }
         } else {
-            if (t_to != t_last) {
+            if (w_to != cnt - 1) {
                 // the first piece of a pair that goes on in the CTAs after this one: theirs, in ascending order
                 const long long pair_end = pos + cnt;
                 // the CTAs after this one whose runs begin inside the pair (with fewer tiles than CTAs some of them are empty)
@@ -1554,16 +1611,18 @@ XR_EXPORT int xr_attention_mma(const void* q, void* out, const void* cache_k, co
                                int hd, int max_pages, int page_size, int window, float scale, int max_seg_len,
                                int max_kv_len, int splits, int any_short, int any_long, const void* cache_base,
                                long long n_pages, int n_layers, int layer, int* status, int* flags, int n_flags,
-                               int uneven, long long row_tiles, const float* sink, float softcap, cudaStream_t stream) {
+                               int uneven, long long row_tiles, const float* sink, float softcap, int keep_first, const float* bias,
+                               int bias_len, cudaStream_t stream) {
     if (n_seg < 1 || H < 1 || K < 1 || H % K != 0 || hd < 16 || hd > 128 || hd % 16 != 0 || page_size < 1 || window < 0 ||
-        (q_stride % 8) != 0 || ((uintptr_t)q & 15) || ((uintptr_t)cache_k & 15) || (page_stride % 8) != 0 || (v_offset % 8) != 0)
+        (q_stride % 8) != 0 || ((uintptr_t)q & 15) || ((uintptr_t)cache_k & 15) || (page_stride % 8) != 0 || (v_offset % 8) != 0 ||
+        keep_first < 0 || (bias != nullptr && (bias_len < 1 || softcap > 0.f)))
         return XR_ERR_ARG;
     if (H / K > 16 && any_short) return XR_ERR_ARG;     // more heads per group than one instruction tile holds
     const int spans = att_spans(max_kv_len, window, (long long)n_seg * K);
     if (any_short && splits < spans) return XR_ERR_ARG;
     AttnMmaArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)cache_k, seg_start, seg_len, seg_pos0,
                   block_tables, part_acc, part_ml, q_stride, page_stride, v_offset, H, K, H / K, max_pages, page_size, window,
-                  spans, 0, scale, -1, n_layers, layer, status, 16, sink, softcap};
+                  spans, 0, scale, -1, n_layers, layer, status, 16, sink, softcap, window > 0 ? keep_first : 0, {bias, bias_len}};
     { long long rows = (long long)(max_seg_len < 1 ? 1 : max_seg_len) * a.G; a.recv_rows = rows < 16 ? (int)rows : 16; }
     a.span = att_choose_span(att_range(max_kv_len, window), (long long)n_seg * K);
     const long long room = (long long)splits * n_seg * K;

@@ -4,6 +4,7 @@
 // position p, head h, kv head h / (H/K):
 //   s_t = (q . k_t) * scale   for t0 <= t <= p,  t0 = max(0, p - window + 1) (0 without a window)
 //   a = softmax(s),  o = sum_t a_t v_t
+// with kept first keys and a bias by distance as options (attention_mask.cuh)
 // (src/model.c:3548-3589; softmax src/model.c:3409-3415).  Keys are taken in
 // chunks of 32 in ascending order with a running maximum, so a query's result
 // depends on its position and the keys only -- not on how the step was cut or
@@ -14,6 +15,7 @@
 // Every token's keys and values, its own included, are read from the cache:
 // the store kernel runs before this one.
 #include "common.cuh"
+#include "attention_mask.cuh"
 #include <math.h>
 
 struct AttnArgs {
@@ -28,6 +30,8 @@ struct AttnArgs {
     float scale;
     const float* sink;           // [H] or null: exp(sink[h]) joins the softmax's denominator once (no key, no value)
     float softcap;               // c > 0: every score becomes c tanh(score / c); 0: scores as they are
+    int keep_first;              // with a window: the first keys that stay visible behind it
+    XrBias bias;
 };
 
 #define AS_MAX_HD 256
@@ -55,9 +59,13 @@ k_attention_simt(AttnArgs a) {
     float m = -INFINITY, l = 0.f;
     const T* kbase = (const T*)a.cache_k;
 
-    for (int k0 = t0; k0 <= pos; k0 += 32) {
+    // the kept keys ahead of the window first, then the window: 32 keys at a time
+    const int kept = min(a.keep_first, t0), kept_chunks = (kept + 31) / 32;
+    const float* bias = a.bias.table != nullptr ? a.bias.table + (size_t)h * a.bias.len : nullptr;
+    for (int c = 0; c < kept_chunks || t0 + 32 * (c - kept_chunks) <= pos; c++) {
+        const int k0 = c < kept_chunks ? 32 * c : t0 + 32 * (c - kept_chunks), end = c < kept_chunks ? kept - 1 : pos;
         int kp = k0 + lane;
-        bool valid = kp <= pos;
+        bool valid = kp <= end;
         long long off = 0;
         float s = -INFINITY;
         if (valid) {
@@ -66,6 +74,7 @@ k_attention_simt(AttnArgs a) {
             const T* kr = kbase + off;
             float dot = 0.f;
             for (int i = 0; i < a.hd; i++) dot = fmaf(qs[warp][i], xr_to_f32<T>(kr[i]), dot);
+            if (bias != nullptr) dot += xr_bias_at(bias, a.bias.len, pos - kp);
             s = dot * a.scale;
             if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
         }
@@ -76,7 +85,7 @@ k_attention_simt(AttnArgs a) {
         l = l * corr + xr_warp_sum(p);
 #pragma unroll
         for (int i = 0; i < ND; i++) acc[i] *= corr;
-        int cnt = min(32, pos - k0 + 1);
+        int cnt = min(32, end - k0 + 1);
         for (int j = 0; j < cnt; j++) {
             float pj = __shfl_sync(0xffffffffu, p, j);
             long long oj = __shfl_sync(0xffffffffu, off, j);
@@ -103,11 +112,12 @@ XR_EXPORT int xr_attention_simt(const void* q, void* out, int dtype, const void*
                                 const int* tok_seg, const int* block_tables, long long page_stride,
                                 long long v_offset, long long q_row_stride, int n, int H, int K, int hd,
                                 int max_pages, int page_size, int window, float scale, const float* sink, float softcap,
-                                cudaStream_t stream) {
-    if (n < 1 || H < 1 || K < 1 || H % K != 0 || hd < 1 || hd > AS_MAX_HD || page_size < 1 || window < 0 || softcap < 0.f)
+                                int keep_first, const float* bias, int bias_len, cudaStream_t stream) {
+    if (n < 1 || H < 1 || K < 1 || H % K != 0 || hd < 1 || hd > AS_MAX_HD || page_size < 1 || window < 0 || softcap < 0.f ||
+        keep_first < 0 || (bias != nullptr && bias_len < 1))
         return XR_ERR_ARG;
     AttnArgs a{q, out, cache_k, positions, tok_seg, block_tables, page_stride, v_offset, q_row_stride,
-               n, H, K, hd, max_pages, page_size, window, scale, sink, softcap};
+               n, H, K, hd, max_pages, page_size, window, scale, sink, softcap, window > 0 ? keep_first : 0, {bias, bias_len}};
     long long warps = (long long)n * H;
     long long blocks = (warps + 3) / 4;
     if (blocks > 0x7fffffffLL) return XR_ERR_ARG;

@@ -26,12 +26,18 @@
 // memory descriptor has leading byte offset = distance between the two 64-column halves and stride byte
 // offset = 8 keys.
 //
+// Kept first keys and a bias by distance are options (attention_mask.cuh).  The bias rows of the CTA's query heads lie in shared
+// memory, one row a head, spaced so that a warp's 32 rows (consecutive tokens of G heads) read 32 banks; a softmax thread adds
+// its row's entry to every raw score it has read from tensor memory.  A tile whose distances all lie beyond the table adds
+// one constant, a tile whose distances all lie inside it reads consecutive entries, others clamp every index.
+//
 // Every wait is bounded; a wait that runs out is recorded in the status word and the CTA runs on (its
 // output is then meaningless) so that all its threads still meet at the barriers and tensor memory is freed.
 //
 // The reference computes prompt attention with one block per (head, token) and a global score scratch
 // (`k_attn`, src/kernels.cu:2043-2141); formulas src/model.c:3548-3589, 3409-3415.
 #include "common.cuh"
+#include "attention_mask.cuh"
 #include <cuda.h>
 #include <math.h>
 
@@ -49,6 +55,9 @@ struct AttnTcArgs {
     int n_seg;
     const float* sink;           // [H] or null: exp(sink[h]) joins the denominator of every softmax of query head h once
     float cap_over_scale, scale_over_cap;   // soft cap c > 0 on the scaled scores: c / scale and scale / c; 0: none
+    int keep_first;              // with a window: the first keys that stay visible behind it
+    XrBias bias;
+    int bias_stride;             // floats between the heads' rows in shared memory; 0: the rows do not fit and are read where they are
 };
 
 __device__ __forceinline__ uint32_t ta_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -157,7 +166,7 @@ __host__ __device__ constexpr uint32_t ta_idesc(bool b_mn, int n) {
 
 // HD: head size, 64 or 128.  Shared memory keeps the layout of head size 128 (a stage of K or V is two halves
 // apart); at head size 64 only the first half of each is filled and read.
-template <int HD>
+template <int HD, bool BIAS>
 __global__ void __launch_bounds__(TA_THREADS, 1)
 k_attention_tc(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map, AttnTcArgs a) {
     // 10 half tiles of 16 KB; the array is declared 1 KB aligned (what the
@@ -185,6 +194,7 @@ k_attention_tc(const __grid_constant__ CUtensorMap q_map, const __grid_constant_
     uint32_t* tmem_slot = (uint32_t*)(bars + 12);
     volatile int* gave_up = (volatile int*)(tmem_slot + 1);
     float* xch = (float*)(tmem_slot + 4);                // [2 tile parities][2 key halves][128 rows]
+    float* bias_s = xch + 2 * 2 * 128;                   // BIAS: [G heads][bias_stride]
 
     // The row tiles of the portions with more than 16 packed rows, laid end to end, are the grid's x (short portions
     // belong to the key-split kernel and have no blocks here: a step may hold dozens of them beside one prompt
@@ -206,13 +216,17 @@ k_attention_tc(const __grid_constant__ CUtensorMap q_map, const __grid_constant_
     const int L = a.seg_len[seg], rows_total = L * a.G;
     const int row0 = tile * TA_ROWS;
     xr_pdl_launch();
+    if (BIAS && a.bias_stride > 0)                       // (constants of the model: no need to wait for the kernel ahead)
+        for (int i = threadIdx.x; i < a.G * a.bias.len; i += TA_THREADS)
+            bias_s[(i / a.bias.len) * a.bias_stride + i % a.bias.len] = a.bias.table[(size_t)kvh * a.G * a.bias.len + i];
     xr_pdl_wait();
     const int pos0 = a.seg_pos0[seg], tok_base = a.seg_start[seg];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int last_row = min(rows_total, row0 + TA_ROWS) - 1;
     const int hi = pos0 + last_row / a.G;
     const int lo = a.window > 0 ? max(0, pos0 + row0 / a.G - a.window + 1) : 0;
-    const int t_lo = lo / TA_KEYS, t_hi = hi / TA_KEYS, n_tiles = t_hi - t_lo + 1;
+    const int t_lo = lo / TA_KEYS, t_hi = hi / TA_KEYS, kept_tiles = xr_kept_tiles(a.keep_first, lo, TA_KEYS);
+    const int n_tiles = kept_tiles + t_hi - t_lo + 1;               // (in the walk's order: xr_walk_tile)
 
     if (threadIdx.x == 0) {
         ta_bar_init(q_full, 1);
@@ -250,7 +264,7 @@ k_attention_tc(const __grid_constant__ CUtensorMap q_map, const __grid_constant_
                 int s = j & 1;
                 if (j >= 2) ta_wait(&empty[s], ((j >> 1) - 1) & 1, gave_up);
                 ta_expect(&full[s], NH * HALF);
-                int key0 = (t_lo + j) * TA_KEYS;
+                int key0 = xr_walk_tile(j, kept_tiles, t_lo) * TA_KEYS;
                 for (int r0 = 0; r0 < TA_KEYS; r0 += box_rows) {
                     int kp = key0 + r0;
                     int pi = kp >> a.page_shift;
@@ -307,12 +321,15 @@ k_attention_tc(const __grid_constant__ CUtensorMap q_map, const __grid_constant_
         const int lo_r = a.window > 0 ? pos - a.window + 1 : 0;
         const uint32_t lane_off = (uint32_t)((warp & 3) * 32) << 16;
         float m = -INFINITY, l = 0.f;          // m: the offset O and l currently carry (log2 domain); l: this thread's half
-        const int pos_first = pos0 + row0 / a.G;                  // smallest position of the CTA's rows
+        const int pos_first = pos0 + row0 / a.G;                  // smallest position of the CTA's rows (the largest: hi)
+        const float* bias = nullptr;                              // this row's bias by distance
+        if (BIAS) bias = a.bias_stride > 0 ? bias_s + (pr % a.G) * a.bias_stride : a.bias.table + (size_t)(kvh * a.G + pr % a.G) * a.bias.len;
         for (int j = 0; j < n_tiles; j++) {
             const uint32_t tm_s = ((j & 1) ? tm_s1 : tm_s0) + lane_off + half * 64;
-            const int key0 = (t_lo + j) * TA_KEYS + half * 64;
+            const int tile0 = xr_walk_tile(j, kept_tiles, t_lo) * TA_KEYS, key0 = tile0 + half * 64;
             // a tile every row sees whole needs no per-score mask
-            const bool masked = a.window > 0 || (t_lo + j) * TA_KEYS + TA_KEYS - 1 > pos_first || row0 + TA_ROWS > rows_total;
+            const bool masked = (a.window > 0 && tile0 <= hi - a.window && tile0 + TA_KEYS > a.keep_first) || tile0 + TA_KEYS - 1 > pos_first ||
+                                row0 + TA_ROWS > rows_total;
             ta_wait(&s_full[j & 1], (j >> 1) & 1, gave_up);
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             // this thread's 64 scores are read once and stay in registers for both passes
@@ -328,13 +345,29 @@ k_attention_tc(const __grid_constant__ CUtensorMap q_map, const __grid_constant_
                     sraw[i] = __float_as_uint(a.cap_over_scale * (1.0f - __fdividef(2.0f, e + 1.0f)));
                 }
             }
+            if (BIAS) {
+                const int d0 = pos - key0, top = a.bias.len - 1;              // distance of the first key; the last key's is d0 - 63
+                const bool dead = pos < 0;
+                if (__all_sync(0xffffffffu, dead || d0 - 63 >= top)) {
+                    const float b = bias[top];
+#pragma unroll
+                    for (int i = 0; i < 64; i++) sraw[i] = __float_as_uint(__uint_as_float(sraw[i]) + b);
+                } else if (a.bias_stride > 0 && __all_sync(0xffffffffu, dead || (d0 >= 63 && d0 <= top))) {
+                    const float* b = bias_s + (pr % a.G) * a.bias_stride + (dead ? 63 : d0);
+#pragma unroll
+                    for (int i = 0; i < 64; i++) sraw[i] = __float_as_uint(__uint_as_float(sraw[i]) + b[-i]);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 64; i++) sraw[i] = __float_as_uint(__uint_as_float(sraw[i]) + xr_bias_at(bias, a.bias.len, d0 - i));
+                }
+            }
             float v[32];
             float mx = -INFINITY;
             if (masked) {
 #pragma unroll
                 for (int i = 0; i < 64; i++) {
                     int kp = key0 + i;
-                    if (kp <= pos && kp >= lo_r) mx = fmaxf(mx, __uint_as_float(sraw[i]));
+                    if (xr_sees(kp, pos, lo_r, a.keep_first)) mx = fmaxf(mx, __uint_as_float(sraw[i]));
                 }
             } else {
                 float m0 = __uint_as_float(sraw[0]), m1 = __uint_as_float(sraw[1]), m2 = __uint_as_float(sraw[2]), m3 = __uint_as_float(sraw[3]);
@@ -392,8 +425,8 @@ k_attention_tc(const __grid_constant__ CUtensorMap q_map, const __grid_constant_
                     float p0 = ta_exp2(fmaf(__uint_as_float(sraw[i]), a.scale_log2, -off));
                     float p1 = ta_exp2(fmaf(__uint_as_float(sraw[i + 1]), a.scale_log2, -off));
                     const int kp = key0 + i;
-                    p0 = (kp <= pos && kp >= lo_r) ? p0 : 0.f;
-                    p1 = (kp + 1 <= pos && kp + 1 >= lo_r) ? p1 : 0.f;
+                    p0 = xr_sees(kp, pos, lo_r, a.keep_first) ? p0 : 0.f;
+                    p1 = xr_sees(kp + 1, pos, lo_r, a.keep_first) ? p1 : 0.f;
                     sum0 += p0; sum1 += p1;
                     __nv_bfloat162 bb = __floats2bfloat162_rn(p0, p1);
                     pall[i >> 1] = *reinterpret_cast<uint32_t*>(&bb);
@@ -404,12 +437,12 @@ k_attention_tc(const __grid_constant__ CUtensorMap q_map, const __grid_constant_
             ta_st32u(((j & 1) ? tm_s1 : tm_s0) + lane_off + half * 32, pall);
             asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
             l += sum0;
-            if ((t_lo + j) * TA_KEYS + TA_KEYS - 1 > hi) {
+            if (tile0 + TA_KEYS - 1 > hi) {
                 // The tile runs past the last key.  Probabilities there are zero, but the value rows hold whatever the
                 // page held before; clear them so that zero times those bytes is zero whatever they are.
                 int s = j & 1;
                 ta_wait(&v_full[s], (j >> 1) & 1, gave_up);
-                int first_bad = hi + 1 - (t_lo + j) * TA_KEYS;
+                int first_bad = hi + 1 - tile0;
                 constexpr int CH = HD / 8;                               // 16-byte chunks of a value row
                 for (int e = half * 128 + r; e < (TA_KEYS - first_bad) * CH; e += 256) {
                     int row = first_bad + e / CH, ch = e % CH;
@@ -492,8 +525,9 @@ XR_EXPORT int xr_attention_tc(const void* q, void* out, const void* cache_base, 
                               const int* seg_pos0, const int* block_tables, int* status, long long q_row_stride, int n,
                               int n_seg, int H, int K, int hd, int max_pages, int page_size, int window, float scale,
                               int max_seg_len, long long row_tiles, long long n_pages, int n_layers, int layer, const float* sink,
-                              float softcap, cudaStream_t stream) {
+                              float softcap, int keep_first, const float* bias, int bias_len, cudaStream_t stream) {
     if (!xr_attention_tc_supported(H, K, hd, page_size) || n < 1 || n_seg < 1 || window < 0 || status == nullptr) return XR_ERR_ARG;
+    if (keep_first < 0 || (bias != nullptr && (bias_len < 1 || softcap > 0.f))) return XR_ERR_ARG;
     if (((uintptr_t)q & 15) || ((uintptr_t)cache_base & 15) || (q_row_stride % 8) != 0) return XR_ERR_ARG;
     const int G = H / K;
     long long total_rows = n_pages * n_layers * 2 * K * page_size;
@@ -532,12 +566,21 @@ XR_EXPORT int xr_attention_tc(const void* q, void* out, const void* cache_base, 
     while ((1 << shift) < page_size) shift++;
     AttnTcArgs a{(__nv_bfloat16*)out, seg_start, seg_len, seg_pos0, block_tables, status, H, K, G, max_pages, page_size, shift,
                  window, n_layers, layer, scale * 1.4426950408889634f, n_seg, sink,
-                 softcap > 0.f ? softcap / scale : 0.f, softcap > 0.f ? scale / softcap : 0.f};
-    constexpr int SMEM = 10 * TA_ROWS * 128 + 128 + 2 * 2 * 128 * 4;
+                 softcap > 0.f ? softcap / scale : 0.f, softcap > 0.f ? scale / softcap : 0.f, window > 0 ? keep_first : 0, {bias, bias_len}, 0};
+    constexpr int SMEM = 10 * TA_ROWS * 128 + 128 + 2 * 2 * 128 * 4, SMEM_MOST = 227 * 1024;
+    int smem = SMEM;
+    if (bias != nullptr) {
+        // rows spaced by 32 / G banks (G heads, 32 / G consecutive tokens a warp), an odd number from 32 heads on
+        const int want = G < 32 ? 32 / G : 1;
+        const int stride = bias_len + ((want - bias_len % 32) + 32) % 32;
+        if (SMEM + (long long)G * stride * 4 <= SMEM_MOST) { a.bias_stride = stride; smem = SMEM + G * stride * 4; }
+    }
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(k_attention_tc<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess ||
-            cudaFuncSetAttribute(k_attention_tc<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess)
+        if (cudaFuncSetAttribute(k_attention_tc<128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess ||
+            cudaFuncSetAttribute(k_attention_tc<64, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess ||
+            cudaFuncSetAttribute(k_attention_tc<128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MOST) != cudaSuccess ||
+            cudaFuncSetAttribute(k_attention_tc<64, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MOST) != cudaSuccess)
             return XR_ERR_LAUNCH;
         configured = true;
     }
@@ -546,7 +589,9 @@ XR_EXPORT int xr_attention_tc(const void* q, void* out, const void* cache_base, 
     long long tiles = row_tiles > 0 ? row_tiles : (((long long)max_seg_len * G + TA_ROWS - 1) / TA_ROWS) * n_seg;
     if (tiles > 0x7fffffffLL) return XR_ERR_ARG;
     const dim3 grid((unsigned)tiles, K, 1);
-    if (hd == 128) xr_launch(k_attention_tc<128>, grid, dim3(TA_THREADS), SMEM, stream, qm, kvm, a);
-    else xr_launch(k_attention_tc<64>, grid, dim3(TA_THREADS), SMEM, stream, qm, kvm, a);
+    if (bias != nullptr && hd == 128) xr_launch((k_attention_tc<128, true>), grid, dim3(TA_THREADS), smem, stream, qm, kvm, a);
+    else if (bias != nullptr) xr_launch((k_attention_tc<64, true>), grid, dim3(TA_THREADS), smem, stream, qm, kvm, a);
+    else if (hd == 128) xr_launch((k_attention_tc<128, false>), grid, dim3(TA_THREADS), smem, stream, qm, kvm, a);
+    else xr_launch((k_attention_tc<64, false>), grid, dim3(TA_THREADS), smem, stream, qm, kvm, a);
     return xr_launch_status();
 }

@@ -17,6 +17,7 @@
 // then make the slot's tail the last taps - 1 inputs.  The walk is token by token, so the state after a token
 // does not depend on how the tokens were cut into steps, bit for bit.
 #include "common.cuh"
+#include "conv_tail.cuh"
 #include <math.h>
 
 #define DL_WARPS 4
@@ -83,27 +84,6 @@ k_delta_prep(const T* __restrict__ proj, long long ldp, const float* __restrict_
         coef[((size_t)t * H + h) * 2] = expf(neg_a[h] * softplus);
         coef[((size_t)t * H + h) * 2 + 1] = 1.0f / (1.0f + expf(-b));
     }
-}
-
-// tail[j] <- the input at place len - (taps - 1) + j of the portion: a row of this step, or, where the portion is
-// shorter than the tail, what the tail held len places further on.  All blocks of the scan that walk a portion share
-// its channels (block `part` of `parts`), after the kernel that read the old tail is complete; a thread reads all of a
-// channel's values before it writes any (eight at a time: the reads of a pass lie ahead of its writes, j ascends).
-template <typename T>
-__device__ __forceinline__ void dl_tail_update(const T* __restrict__ proj, long long ldp, float* tail, int start, int len,
-                                               int CH, int taps, int part, int parts) {
-    for (int c = part * blockDim.x + threadIdx.x; c < CH; c += parts * blockDim.x)
-        for (int j0 = 0; j0 < taps - 1; j0 += 8) {
-            float x[8];
-#pragma unroll
-            for (int i = 0; i < 8; i++) {
-                const int j = j0 + i, src = len - (taps - 1) + j;
-                x[i] = j >= taps - 1 ? 0.f : (src >= 0 ? xr_to_f32<T>(proj[(size_t)(start + src) * ldp + c]) : tail[(size_t)(j + len) * CH + c]);
-            }
-#pragma unroll
-            for (int i = 0; i < 8; i++)
-                if (j0 + i < taps - 1) tail[(size_t)(j0 + i) * CH + c] = x[i];
-        }
 }
 
 // LPC lanes (8 or 16) share a value column.  Thread (column, row lane l) keeps RPT rows of its column, four at a time:
@@ -239,7 +219,7 @@ k_delta_scan(const float* __restrict__ qkv, const float* __restrict__ coef, floa
     }
     xr_pdl_launch();
     if (taps > 1)
-        dl_tail_update<T>(proj, ldp, state + (size_t)slot * state_stride + (size_t)H * V * D, start, len, CH, taps,
+        xr_tail_update<T>(proj, ldp, state + (size_t)slot * state_stride + (size_t)H * V * D, start, len, CH, taps,
                           blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
 }
 

@@ -376,6 +376,9 @@ XR_EXPORT int xr_rmsnorm_act(const void* in, int dtype, long long ld_in, const f
 // float64, cosine and sine in float32).  The attention kernels take one head size hd >= max(D, Vd) for keys and
 // values: Q goes to q_out [n, q_ld] (head h at h * hd), K and V to the token's cache rows, each head filled up to hd
 // with zeros, which change neither a score nor a sum.  One block per token, a warp per head.
+//
+// Value mixing (v_first, [n][K][Vd] rows of this step): with v_mix 1 the layer leaves its values there; with v_mix 2 what is cached
+// is (1 - v_lambda) v + v_lambda v_first, in float32 before the rounding to the cache.
 // ---------------------------------------------------------------------------
 struct QkNormStoreArgs {
     const void* in;
@@ -401,7 +404,18 @@ struct QkNormStoreArgs {
     const float* partial; const float* bias; int splits, cols, n;
     float mscale;                // factor on every cosine and sine
     int norm_after;              // the unit norm is taken of the ROTATED head (with mscale other than one the order matters)
+    void* v_first; int v_mix;    // values that layers share: 0 no mixing, 1 this layer leaves its own, 2 it mixes them in
+    float v_lambda;
 };
+
+// One value element (column i of the token's K * Vd) on its way to the cache.
+template <typename T>
+__device__ __forceinline__ T qk_mix_value(const QkNormStoreArgs& a, int t, int i, T v) {
+    if (a.v_mix == 0) return v;
+    T* first = (T*)a.v_first + (size_t)t * a.K * a.Vd + i;
+    if (a.v_mix == 1) { *first = v; return v; }
+    return xr_from_f32<T>((1.0f - a.v_lambda) * xr_to_f32<T>(v) + a.v_lambda * xr_to_f32<T>(*first));
+}
 
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -528,14 +542,14 @@ k_qk_norm_rope_store(QkNormStoreArgs a) {
         for (int i = first * blockDim.x + threadIdx.x; i < behind + n_v; i += step) {
             if (i < behind) { finished(v_at + a.K * a.Vd + i); continue; }
             const int kvh = (i - behind) / a.hd, e = (i - behind) % a.hd;
-            vdst[(size_t)kvh * head_step + e] = e < a.Vd ? finished(v_at + kvh * a.Vd + e) : xr_from_f32<T>(0.f);
+            vdst[(size_t)kvh * head_step + e] = e < a.Vd ? qk_mix_value<T>(a, t, kvh * a.Vd + e, finished(v_at + kvh * a.Vd + e)) : xr_from_f32<T>(0.f);
         }
         return;
     }
     if (kdst == nullptr) return;
     T* vdst = kdst + a.v_offset;
     const T* vsrc = row + (size_t)v_at;
-    if (pairs && !(a.Vd & 1) && !(a.v_offset & 1) && !(((a.H + a.K) * a.D) & 1)) {
+    if (pairs && a.v_mix == 0 && !(a.Vd & 1) && !(a.v_offset & 1) && !(((a.H + a.K) * a.D) & 1)) {
         const int hd2 = a.hd >> 1;
         for (int i = threadIdx.x; i < a.K * hd2; i += blockDim.x) {
             const int kvh = i / hd2, e = (i % hd2) * 2;
@@ -547,7 +561,7 @@ k_qk_norm_rope_store(QkNormStoreArgs a) {
     }
     for (int i = threadIdx.x; i < a.K * a.hd; i += blockDim.x) {
         const int kvh = i / a.hd, e = i % a.hd;
-        vdst[(size_t)kvh * head_step + e] = e < a.Vd ? vsrc[(size_t)kvh * a.Vd + e] : xr_from_f32<T>(0.f);
+        vdst[(size_t)kvh * head_step + e] = e < a.Vd ? qk_mix_value<T>(a, t, kvh * a.Vd + e, vsrc[(size_t)kvh * a.Vd + e]) : xr_from_f32<T>(0.f);
     }
 }
 
@@ -662,7 +676,21 @@ k_qk_norm_rope_store_vec(QkNormStoreArgs a) {
         Bf16x8 v;
 #pragma unroll
         for (int k = 0; k < 4; k++) v.p[k] = __floats2bfloat162_rn(0.f, 0.f);
-        if (e < a.Vd) v = *reinterpret_cast<const Bf16x8*>(row + (size_t)v_at + (size_t)kvh * a.Vd + e);
+        if (e < a.Vd) {
+            v = *reinterpret_cast<const Bf16x8*>(row + (size_t)v_at + (size_t)kvh * a.Vd + e);
+            if (a.v_mix != 0) {
+                Bf16x8* first = reinterpret_cast<Bf16x8*>((__nv_bfloat16*)a.v_first + (size_t)t * a.K * a.Vd + (size_t)kvh * a.Vd + e);
+                if (a.v_mix == 1) *first = v;
+                else {
+                    const Bf16x8 f = *first;
+#pragma unroll
+                    for (int k = 0; k < 4; k++) {
+                        const float2 x = __bfloat1622float2(v.p[k]), y = __bfloat1622float2(f.p[k]);
+                        v.p[k] = __floats2bfloat162_rn((1.0f - a.v_lambda) * x.x + a.v_lambda * y.x, (1.0f - a.v_lambda) * x.y + a.v_lambda * y.y);
+                    }
+                }
+            }
+        }
         *reinterpret_cast<Bf16x8*>(vdst + (size_t)kvh * head_step + e) = v;
     }
 }
@@ -672,7 +700,8 @@ XR_EXPORT int xr_qk_norm_rope_store(const void* in, int dtype, long long ld_in, 
                                     void* cache_k, long long page_stride, long long v_offset, int n, int H, int K, int D, int Vd, int hd,
                                     int rotary_dim, int max_pages, int page_size, int adjacent_pairs, float eps, int unit_norm,
                                     float q_coef, int q_every, const float* partial, int splits, const float* bias, int cols,
-                                    float mscale, int norm_after, cudaStream_t stream) {
+                                    float mscale, int norm_after, void* v_first, int v_mix, float v_lambda, cudaStream_t stream) {
+    if (v_mix < 0 || v_mix > 2 || (v_mix != 0 && (v_first == nullptr || cache_k == nullptr || ((uintptr_t)v_first & 15)))) return XR_ERR_ARG;
     if (partial != nullptr && (splits < 1 || D > 256 || cols < (H + K) * D + K * Vd || cols > ld_in)) return XR_ERR_ARG;
     if (n < 1 || H < 1 || K < 1 || D < 1 || Vd < 1 || hd < D || hd < Vd || rotary_dim < 0 || rotary_dim > D || (rotary_dim & 1) ||
         page_size < 1 || (rotary_dim > 0 && freq == nullptr) || (q_w == nullptr) != (k_w == nullptr) || q_every < 0 ||
@@ -681,7 +710,7 @@ XR_EXPORT int xr_qk_norm_rope_store(const void* in, int dtype, long long ld_in, 
     const int pairs = !((D | hd | ld_in | q_ld | page_stride) & 1) && !(((uintptr_t)in | (uintptr_t)q_out | (uintptr_t)cache_k) & 3);
     QkNormStoreArgs a{in, ld_in, q_out, q_ld, positions, tok_seg, block_tables, freq, q_w, k_w, cache_k, page_stride, v_offset,
                       H, K, D, Vd, hd, rotary_dim, max_pages, page_size, adjacent_pairs ? 1 : 0, eps, pairs, unit_norm ? 1 : 0,
-                      q_coef, q_every, partial, bias, splits, cols, n, mscale, norm_after ? 1 : 0};
+                      q_coef, q_every, partial, bias, splits, cols, n, mscale, norm_after ? 1 : 0, v_first, v_mix, v_lambda};
     const size_t smem = ((size_t)rotary_dim + 8 * (size_t)D) * sizeof(float);
     if (smem > 48 * 1024) return XR_ERR_ARG;
     // bfloat16 rows of whole prompts whose sizes, strides and addresses all fall on 16-byte borders: eight elements a lane
@@ -716,11 +745,12 @@ XR_EXPORT int xr_qk_norm_rope_store(const void* in, int dtype, long long ld_in, 
 // (src/model.c:4425-4452, `gated_act`); ungated, h = act(x) of x [n, F] (src/model.c:6380-6396).
 // act 1: SiLU, g / (1 + exp(-g)), 0 for g < -80 (src/model.c:4451-4452; the reference's kernel is
 // src/kernels.cu:2868-2874); act 2: tanh-GELU, 0.5 g (1 + tanh(0.7978845608 (g + 0.044715 g^3)))
-// (src/model.c:4438-4441); act 0: none.  Full-precision expf and tanhf: this is the kernel of the true 32-bit path.
+// (src/model.c:4438-4441); act 4: the square of relu; act 0: none.  Full-precision expf and tanhf: this is the kernel of the true 32-bit path.
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ float xr_activation(int act, float g) {
     if (act == 1) return g < -80.0f ? 0.0f : g / (1.0f + expf(-g));
     if (act == 2) return 0.5f * g * (1.0f + tanhf(0.7978845608f * (g + 0.044715f * g * g * g)));
+    if (act == 4) { const float r = fmaxf(g, 0.f); return r * r; }
     return g;
 }
 
@@ -750,7 +780,7 @@ __global__ void k_act_mul(const T* gu, T* h, int n, int F, int act, int gated, f
 
 // gated: gu [n, 2F] -> h [n, F]; ungated: gu [n, F] -> h [n, F] (h may be gu)
 XR_EXPORT int xr_act_mul(const void* gu, void* h, int dtype, int n, int F, int act, int gated, float limit, cudaStream_t stream) {
-    if (n < 1 || F < 1 || act < 0 || act > 3 || (act == 3 && !gated)) return XR_ERR_ARG;
+    if (n < 1 || F < 1 || act < 0 || act > 4 || (act == 3 && !gated)) return XR_ERR_ARG;
     size_t total = (size_t)n * F;
     int blocks = (int)((total + 255) / 256 < (size_t)xr_sm_count() * 16 ? (total + 255) / 256 : xr_sm_count() * 16);
     if (dtype == XR_F32) xr_launch((k_act_mul<float>), dim3(blocks), dim3(256), 0, stream, (const float*)gu, (float*)h, n, F, act, gated, limit);

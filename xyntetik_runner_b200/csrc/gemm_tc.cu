@@ -50,6 +50,7 @@ __host__ __device__ constexpr int tc_threads(int bn) { return bn <= 16 ? 192 : T
 #define TC_ACT_SILU 1
 #define TC_ACT_GELU_TANH 2
 #define TC_ACT_SWISH_CLAMP 3     // gated products only, see tc_gate
+#define TC_ACT_RELU2 4           // the square of relu
 
 // ---------------------------------------------------------------------------------------------
 // PTX wrappers
@@ -122,6 +123,7 @@ __device__ __forceinline__ float tc_gelu_tanh(float g) {
     return 0.5f * g * (1.0f + t);
 }
 __device__ __forceinline__ float tc_act(int act, float g) {
+    if (act == TC_ACT_RELU2) { const float r = fmaxf(g, 0.f); return r * r; }
     return act == TC_ACT_SILU ? tc_silu(g) : (act == TC_ACT_GELU_TANH ? tc_gelu_tanh(g) : g);
 }
 // What a gated product stores for a feature with gate sum g and up sum u: act(g) * u, or for TC_ACT_SWISH_CLAMP
@@ -814,7 +816,7 @@ XR_EXPORT int xr_gemm_tc(const void* X, const void* W, const float* bias, void* 
     if (epilogue == TC_EPI_ADD && (out_dtype != XR_F32 || act != TC_ACT_NONE)) return XR_ERR_ARG;
     if (out_dtype != XR_F32 && out_dtype != XR_BF16) return XR_ERR_ARG;
     const bool gated = epilogue == TC_EPI_GATED;
-    if (act != TC_ACT_NONE && act != TC_ACT_SILU && act != TC_ACT_GELU_TANH && !(act == TC_ACT_SWISH_CLAMP && gated)) return XR_ERR_ARG;
+    if (act != TC_ACT_NONE && act != TC_ACT_SILU && act != TC_ACT_GELU_TANH && act != TC_ACT_RELU2 && !(act == TC_ACT_SWISH_CLAMP && gated)) return XR_ERR_ARG;
     if (gated && (!w_packed || bias != nullptr)) return XR_ERR_ARG;
     const TcPlan pl = plan_product(n, n_out, K, gated, force_splits, defer_finish != 0, scratch ? scratch_floats : 0);
     CUtensorMap mw, mx;
@@ -871,7 +873,7 @@ XR_EXPORT int xr_gemm_tc_grouped(const void* X, const void* W, void* out, int ou
     if (epilogue != TC_EPI_STORE && epilogue != TC_EPI_GATED) return XR_ERR_ARG;
     if (out_dtype != XR_F32 && out_dtype != XR_BF16) return XR_ERR_ARG;
     const bool gated = epilogue == TC_EPI_GATED;
-    if (act != TC_ACT_NONE && act != TC_ACT_SILU && act != TC_ACT_GELU_TANH && !(act == TC_ACT_SWISH_CLAMP && gated)) return XR_ERR_ARG;
+    if (act != TC_ACT_NONE && act != TC_ACT_SILU && act != TC_ACT_GELU_TANH && act != TC_ACT_RELU2 && !(act == TC_ACT_SWISH_CLAMP && gated)) return XR_ERR_ARG;
     const int row_tiles = gated ? (n_out + 63) / 64 : (n_out + TC_BM - 1) / TC_BM;
     const int total_kb = (K + TC_BK - 1) / TC_BK;
     const int tok_tiles = n / bn;

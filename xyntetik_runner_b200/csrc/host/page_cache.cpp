@@ -7,7 +7,8 @@
 // reference's per-layer sliding flag, src/model.h:229-235).  Every group has a pool of pages of its own and every
 // request slot a row of page numbers per group (the block table, -1 where no page is held).  Pages go back to
 // their pool when a request ends and, in a window group, as soon as every position in the page lies behind the
-// window of every query still to come.  The block tables live in memory that the caller owns (numpy arrays), so
+// window of every query still to come -- except the pages that hold the first `keep` positions, where the layers of the
+// group go on seeing a request's first tokens from anywhere: those stay until the request ends.  The block tables live in memory that the caller owns (numpy arrays), so
 // that the engine copies rows of them into the step description without asking this library.
 //
 // A request is known here by its slot.  Return codes: XRH_OK, or one of the errors below; nothing is changed
@@ -52,12 +53,13 @@ struct Request {
     bool open = false;
     long long length = 0;             // tokens whose keys are in the cache
     long long reserved = 0;           // tokens reserved beyond `length` for the step in flight
-    std::vector<int> first_live;      // per group: table entries below this were released
+    std::vector<int> first_live;      // per group: table entries below this were released (but for the kept first pages)
 };
 
 struct Cache {
     int groups, page_size, max_requests, max_pages;
     std::vector<int> window;          // per group, < 0: every key is kept
+    std::vector<int> kept;            // per group: pages from a request's start that stay whatever the window has passed
     std::vector<Pool> pools;
     std::vector<int32_t*> tables;     // per group [max_requests][max_pages], owned by the caller
     std::vector<Request> reqs;
@@ -89,12 +91,17 @@ struct Cache {
             out[g] = (int)(want_upto > lo ? want_upto - lo : 0);
         }
     }
+    // table entries below first_live may still hold pages: the kept ones
+    long long first_to_release(const Request& r, int g) const {
+        long long a = r.first_live[(size_t)g], b = kept[(size_t)g];
+        return a > b ? a : b;
+    }
     // pages that the window lets go before a query at the request's next position
     long long releasable(const Request& r, int g) const {
         long long pos = r.length + r.reserved;
         long long first = first_needed_page(g, pos), held_upto = ceil_pages(pos);
         long long upto = first < held_upto ? first : held_upto;
-        long long n = upto - r.first_live[(size_t)g];
+        long long n = upto - first_to_release(r, g);
         return n > 0 ? n : 0;
     }
     bool can_reserve(const Request& r, long long n_new) const {
@@ -112,7 +119,7 @@ struct Cache {
             long long first = first_needed_page(g, pos), held_upto = ceil_pages(pos);
             if (held_upto < first) first = held_upto;
             int32_t* tab = row(g, slot);
-            for (long long i = r.first_live[(size_t)g]; i < first; i++)
+            for (long long i = first_to_release(r, g); i < first; i++)
                 if (tab[i] >= 0) {
                     pools[(size_t)g].give(tab[i]);
                     tab[i] = -1;
@@ -134,15 +141,17 @@ XRH_EXPORT int xrh_pool_take(void* p) { return ((Pool*)p)->take(); }            
 XRH_EXPORT int xrh_pool_give(void* p, int page) { return ((Pool*)p)->give(page) ? XRH_OK : XRH_NOT_HELD; }
 
 // ---- the cache manager -------------------------------------------------------------------------------------
-// windows[g] < 0: group g keeps every key.  tables[g]: int32 [max_requests][max_pages], filled with -1 here.
-XRH_EXPORT void* xrh_cache_create(int groups, const int* windows, int n_pages, int page_size, int max_requests, int max_pages,
-                                  int32_t** tables) {
+// windows[g] < 0: group g keeps every key.  keep_first[g]: positions from a request's start that stay in group g behind its
+// window (null: none anywhere).  tables[g]: int32 [max_requests][max_pages], filled with -1 here.
+XRH_EXPORT void* xrh_cache_create(int groups, const int* windows, const int* keep_first, int n_pages, int page_size, int max_requests,
+                                  int max_pages, int32_t** tables) {
     if (groups < 0 || n_pages < 1 || page_size < 1 || max_requests < 1 || max_pages < 1) return nullptr;
     Cache* c = new (std::nothrow) Cache();
     if (!c) return nullptr;
     c->groups = groups; c->page_size = page_size; c->max_requests = max_requests; c->max_pages = max_pages;
     for (int g = 0; g < groups; g++) {
         c->window.push_back(windows[g]);
+        c->kept.push_back(keep_first != nullptr && keep_first[g] > 0 ? (int)c->ceil_pages(keep_first[g]) : 0);
         c->pools.emplace_back(n_pages);
         c->tables.push_back(tables[g]);
         c->high_water.push_back(0);
@@ -180,7 +189,7 @@ XRH_EXPORT int xrh_close(void* h, int slot) {
     long long upto = c->ceil_pages(r->length + r->reserved);
     for (int g = 0; g < c->groups; g++) {
         int32_t* tab = c->row(g, slot);
-        for (long long i = r->first_live[(size_t)g]; i < upto; i++)
+        for (long long i = 0; i < upto; i++)
             if (tab[i] >= 0) c->pools[(size_t)g].give(tab[i]);
         for (int i = 0; i < c->max_pages; i++) tab[i] = -1;
     }
@@ -285,7 +294,7 @@ XRH_EXPORT int xrh_audit(void* h, char* msg, int cap) {
             }
             long long upto = c->ceil_pages(r.length + r.reserved);
             for (int i = 0; i < c->max_pages; i++) {
-                bool live = r.first_live[(size_t)g] <= i && i < upto;
+                bool live = (r.first_live[(size_t)g] <= i || i < c->kept[(size_t)g]) && i < upto;
                 if (tab[i] >= 0) {
                     if (!live) FAIL("group %d slot %d: page at index %d outside its live range", g, s, i);
                     if (tab[i] >= pool.n_pages) FAIL("group %d slot %d: page number at index %d is outside the pool", g, s, i);

@@ -3,6 +3,9 @@
 //
 //   z = W_router h (float32, a product of the caller);  the `top` largest z are chosen (ties: the lower index),
 //   weights = softmax over the chosen z only;  out[t] += sum_j weight_j * expert_{e_j}(h[t]).
+// Other scores, a correction of the choice, groups of experts and a factor on the weights: see k_route_topk and k_route_groups.
+// The router may have more outputs than there are experts: the outputs from E on are identity experts, whose output is h[t]
+// itself.  They take part in the choice, have no rows in the plan (pair_row -1), and the weighted sum adds weight * h[t] for them.
 // An expert is a gated feed-forward: y = gate_act(W_gate h, W_up h), then W_down y (see xr_gate below for the
 // activations).  No step reads anything back to the host: the plan of who computes what is made on the device, and
 // the grids are sized for the worst case (every tile index beyond the plan's count returns at once).
@@ -64,11 +67,94 @@ XR_EXPORT int xr_route_topk(const float* z, int* ids, float* wts, int n, int E, 
 }
 
 // ---------------------------------------------------------------------------------------------
+// Choice with scores s = softmax(z) over ALL outputs and by groups: E outputs in `groups` equal groups of neighbours; the choice goes
+// by c = s + correction (null: s); a group's score is its largest c, the `keep` best groups (ties: the lower index) stay and the
+// `top` largest c inside them are chosen; weights s * scale, not renormalised.  One warp per token, c in shared memory.
+// ---------------------------------------------------------------------------------------------
+#define ROUTE_MAX_E 1024
+
+__device__ __forceinline__ void route_argmax(float& v, int& i) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, i, o);
+        if (ov > v || (ov == v && oi < i)) { v = ov; i = oi; }
+    }
+}
+
+__global__ void __launch_bounds__(128)
+k_route_groups(const float* __restrict__ z, int* __restrict__ ids, float* __restrict__ wts, int n, int E, int top,
+               const float* __restrict__ correction, int groups, int keep, float scale) {
+    xr_pdl_launch();
+    extern __shared__ float route_sm[];                            // per warp: c [E], the groups' scores [groups], then the groups kept [groups]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 4 + warp, per = E / groups;
+    if (t >= n) return;
+    float* c = route_sm + (size_t)warp * (E + 2 * groups);
+    float* best = c + E;
+    float* stays = best + groups;
+    xr_pdl_wait();
+    const float* row = z + (size_t)t * E;
+    float m = -INFINITY, sum = 0.f;
+    for (int e = lane; e < E; e += 32) m = fmaxf(m, row[e]);
+    m = xr_warp_max(m);
+    for (int e = lane; e < E; e += 32) sum += expf(row[e] - m);
+    sum = xr_warp_sum(sum);
+    for (int e = lane; e < E; e += 32) c[e] = expf(row[e] - m) / sum + (correction != nullptr ? correction[e] : 0.f);
+    __syncwarp();
+    if (groups > 1) {
+        for (int g = lane; g < groups; g += 32) {
+            float b = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; e++) b = fmaxf(b, c[e]);
+            best[g] = b;
+            stays[g] = 0.f;
+        }
+        __syncwarp();
+        for (int k = 0; k < keep; k++) {
+            float bv = -INFINITY;
+            int bg = 0x7fffffff;
+            for (int g = lane; g < groups; g += 32)
+                if (stays[g] == 0.f && (bg == 0x7fffffff || best[g] > bv)) { bv = best[g]; bg = g; }
+            route_argmax(bv, bg);
+            if (lane == 0 && bg < groups) stays[bg] = 1.f;
+            __syncwarp();
+        }
+        for (int e = lane; e < E; e += 32)
+            if (stays[e / per] == 0.f) c[e] = -INFINITY;
+        __syncwarp();
+    }
+    for (int j = 0; j < top; j++) {
+        float bv = -INFINITY;
+        int be = 0x7fffffff;
+        for (int e = lane; e < E; e += 32)
+            if (c[e] > bv) { bv = c[e]; be = e; }
+        route_argmax(bv, be);
+        if (be >= E) be = 0;                                       // (nothing left to choose: scores that are no numbers)
+        if (lane == 0) {
+            ids[(size_t)t * top + j] = be;
+            wts[(size_t)t * top + j] = expf(row[be] - m) / sum * scale;
+            c[be] = -INFINITY;
+        }
+        __syncwarp();
+    }
+}
+
+// E: outputs of the router, identity experts included.  groups 1 (keep 1): no groups.
+XR_EXPORT int xr_route_groups(const float* z, int* ids, float* wts, int n, int E, int top, const float* correction, int groups, int keep,
+                              float scale, cudaStream_t stream) {
+    if (n < 1 || E < 1 || E > ROUTE_MAX_E || groups < 1 || E % groups || keep < 1 || keep > groups || top < 1 || top > keep * (E / groups))
+        return XR_ERR_ARG;
+    const size_t smem = 4 * (size_t)(E + 2 * groups) * sizeof(float);
+    if (smem > 48 * 1024) return XR_ERR_ARG;
+    xr_launch(k_route_groups, dim3((n + 3) / 4), dim3(128), smem, stream, z, ids, wts, n, E, top, correction, groups, keep, scale);
+    return xr_launch_status();
+}
+
+// ---------------------------------------------------------------------------------------------
 // Plan, one block: rows = the n * top pairs sorted by expert, every expert's rows starting at a multiple of `align`
 // (the row tile of the kernel that multiplies them), so that a tile of `align` rows meets one expert.
 //   row_src [max_rows]: the pair (t * top + j) that row r computes, -1 for a row of padding;
 //   pair_row [pairs]: the row of every pair;  tile_group [max_rows / align]: the tile's expert, -1 for a tile without rows.
-//   max_rows = (pairs / align + E + 1) * align always suffices.
+//   max_rows = (pairs / align + E + 1) * align always suffices.  A pair whose id is E or more (an identity expert) has no row.
 // Which row a pair gets among its expert's rows depends on the order in which threads arrive; a row's result does not.
 // ---------------------------------------------------------------------------------------------
 #define MOE_MAX_E 1024
@@ -81,7 +167,10 @@ k_moe_plan(const int* __restrict__ ids, int* __restrict__ row_src, int* __restri
     for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
     xr_pdl_wait();
     __syncthreads();
-    for (int p = threadIdx.x; p < pairs; p += blockDim.x) atomicAdd(&count[ids[p]], 1);
+    for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
+        const int e = ids[p];
+        if (e < E) atomicAdd(&count[e], 1);
+    }
     __syncthreads();
     if (threadIdx.x == 0) {
         int tiles = 0;
@@ -99,7 +188,9 @@ k_moe_plan(const int* __restrict__ ids, int* __restrict__ row_src, int* __restri
     for (int e = threadIdx.x; e < E; e += blockDim.x)
         for (int t = tile0[e]; t < tile0[e + 1]; t++) tile_group[t] = e;
     for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
-        const int r = atomicAdd(&cursor[ids[p]], 1);
+        const int e = ids[p];
+        if (e >= E) { pair_row[p] = -1; continue; }
+        const int r = atomicAdd(&cursor[e], 1);
         row_src[r] = p;
         pair_row[p] = r;
     }
@@ -163,6 +254,7 @@ __device__ __forceinline__ float moe_gate(int act, float limit, float g, float u
     }
     if (act == 1) return (g < -80.0f ? 0.0f : g / (1.0f + expf(-g))) * u;
     if (act == 2) return 0.5f * g * (1.0f + tanhf(0.7978845608f * (g + 0.044715f * g * g * g))) * u;
+    if (act == 4) { const float r = fmaxf(g, 0.f); return r * r * u; }
     return g * u;
 }
 
@@ -238,7 +330,7 @@ k_moe_gemm(const TA* __restrict__ A, long long lda, const TW* __restrict__ W, TO
 XR_EXPORT int xr_moe_gemm(const void* A, int a_dtype, long long lda, const void* W, int w_dtype, void* out, int out_dtype,
                           long long ldo, const int* row_src, const int* tile_group, int max_tiles,
                           int top, int N, int K, int gated, int act, float limit, cudaStream_t stream) {
-    if (max_tiles < 1 || N < 1 || K < 1 || top < 1 || act < 0 || act > 3) return XR_ERR_ARG;
+    if (max_tiles < 1 || N < 1 || K < 1 || top < 1 || act < 0 || act > 4) return XR_ERR_ARG;
     const int cols = gated ? 32 : 64;
     dim3 grid(max_tiles, (N + cols - 1) / cols);
     if (grid.y > 65535) return XR_ERR_ARG;
@@ -260,27 +352,40 @@ XR_EXPORT int xr_moe_gemm(const void* A, int a_dtype, long long lda, const void*
 }
 
 // ---------------------------------------------------------------------------------------------
-// d[t][c] += sum_j wts[t][j] * Z[pair_row[t * top + j]][c], j ascending (float32).
+// d[t][c] += sum_j wts[t][j] * Z[pair_row[t * top + j]][c], j ascending (float32).  A pair without a row (pair_row -1) is an identity
+// expert's: its term is wts[t][j] * h[t][c].
 // ---------------------------------------------------------------------------------------------
+template <typename T>
 __global__ void __launch_bounds__(256)
 k_moe_combine(float* __restrict__ d, const float* __restrict__ Z, const float* __restrict__ wts, const int* __restrict__ pair_row,
-              int n, int width, int top) {
+              const T* __restrict__ h, long long ldh, int n, int width, int top) {
     xr_pdl_launch();
     xr_pdl_wait();
     const size_t total = (size_t)n * width;
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
         const size_t t = i / width, c = i % width;
         float s = 0.f;
-        for (int j = 0; j < top; j++) s = fmaf(wts[t * top + j], Z[(size_t)pair_row[t * top + j] * width + c], s);
+        for (int j = 0; j < top; j++) {
+            const int r = pair_row[t * top + j];
+            float v = 0.f;
+            if (r >= 0) v = Z[(size_t)r * width + c];
+            else if (h != nullptr) v = xr_to_f32<T>(h[t * ldh + c]);
+            s = fmaf(wts[t * top + j], v, s);
+        }
         d[i] += s;
     }
 }
 
-XR_EXPORT int xr_moe_combine(float* d, const float* Z, const float* wts, const int* pair_row, int n, int width, int top,
-                             cudaStream_t stream) {
-    if (n < 1 || width < 1 || top < 1) return XR_ERR_ARG;
+// h [n][ldh] in h_dtype: what the experts read, for identity experts; null: there are none.
+XR_EXPORT int xr_moe_combine(float* d, const float* Z, const float* wts, const int* pair_row, const void* h, int h_dtype, long long ldh, int n,
+                             int width, int top, cudaStream_t stream) {
+    if (n < 1 || width < 1 || top < 1 || (h != nullptr && ldh < width)) return XR_ERR_ARG;
     const size_t total = (size_t)n * width;
     int blocks = (int)((total + 255) / 256 < (size_t)xr_sm_count() * 16 ? (total + 255) / 256 : xr_sm_count() * 16);
-    xr_launch(k_moe_combine, dim3(blocks), dim3(256), 0, stream, d, Z, wts, pair_row, n, width, top);
+    if (h == nullptr || h_dtype == XR_F32)
+        xr_launch((k_moe_combine<float>), dim3(blocks), dim3(256), 0, stream, d, Z, wts, pair_row, (const float*)h, ldh, n, width, top);
+    else if (h_dtype == XR_BF16)
+        xr_launch((k_moe_combine<__nv_bfloat16>), dim3(blocks), dim3(256), 0, stream, d, Z, wts, pair_row, (const __nv_bfloat16*)h, ldh, n, width, top);
+    else return XR_ERR_ARG;
     return xr_launch_status();
 }

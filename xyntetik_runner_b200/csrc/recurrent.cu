@@ -1,4 +1,4 @@
-// Two linear recurrences with a fixed-size float32 state per request slot.
+// Three linear recurrences with a fixed-size float32 state per request slot.
 //
 // (1) The real-gated linear recurrent unit (the recurrence of Griffin's recurrent block).  With R channels in B blocks of
 //     R / B, a short causal convolution per channel, and per token the projections' rows y' and x' (float32, biases included):
@@ -16,9 +16,16 @@
 //       S <- decay_h S + k v^T,   o = S^T q,   q, k, v the projections' rows behind their activation.
 //     k_decay_scan, a warp per eight value columns of a head: the state in registers, see there.
 //
-// Everything here is float32 in both precisions, and both walks go token by token: the state after a token does not depend
+// (3) The state-space dual recurrence of Mamba-2: S [N][V] per head, head h reading key and query rows B, C of group h / (H / G),
+//       S <- exp(-exp(A_log_h) dt) S + dt B x^T,   y = S^T C + D_h x,   dt = softplus(dt' + dt_bias_h)
+//     with x, B, C behind a short causal convolution per channel (bias) and silu.  k_ssd_prep: the convolution and the two numbers
+//     per token and head (decay, dt); the walk is k_decay_scan's with those in place of a constant decay.  State per slot:
+//     S [H][V][N], then the last taps - 1 inputs of the convolution [taps-1][H V + 2 G N].
+//
+// Everything here is float32 in both precisions, and the walks go token by token: the state after a token does not depend
 // on how the tokens were cut into steps, bit for bit.
 #include "common.cuh"
+#include "conv_tail.cuh"
 #include <math.h>
 
 #define RG_MAX_TAPS 16
@@ -303,7 +310,18 @@ XR_EXPORT int xr_rglru(float* proj, long long ldp, int y_col, int x_col, const f
 // registers before this chunk is walked and stored behind it (16 bytes a load where sizes and addresses allow: VEC).  A step of
 // many tokens applies silu to the rows beforehand, in
 // place (k_silu_cols); a step of few applies it on the way into shared memory.
+// SSD: the decay and the factor on the value come per token and head (coef), heads share key and query rows by `rep`, the
+// value times skip[h] joins the read-out, a column's state lies together in memory ([H][V][D] instead of [H][D][V]), and the
+// blocks of a portion leave the convolution's new tail behind the walk.
 #define DA_WARPS 8
+
+struct SsdArgs {
+    const float* coef;           // [n][H][2]: decay, dt
+    const float* skip;           // [H]
+    const float* raw;            // the convolution's inputs, row stride ld_raw, CH columns
+    long long ld_raw;
+    int CH, taps, rep;
+};
 
 __global__ void k_silu_cols(float* __restrict__ rows, long long ld, int cols, size_t total) {
     xr_pdl_launch();
@@ -314,35 +332,64 @@ __global__ void k_silu_cols(float* __restrict__ rows, long long ld, int cols, si
     }
 }
 
-template <int JD, int VC, int CH, bool VEC>
+template <int JD, int VC, int CH, bool VEC, bool SSD>
 __global__ void __launch_bounds__(32 * DA_WARPS)
 k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col, int v_col, const float* __restrict__ decay,
              float* __restrict__ state, long long state_stride, const int* __restrict__ seg_start, const int* __restrict__ seg_len,
-             const int* __restrict__ seg_slot, float* __restrict__ o, int H, int D, int V, int activated) {
+             const int* __restrict__ seg_slot, float* __restrict__ o, int H, int D, int V, int activated, SsdArgs ssd) {
     xr_pdl_launch();
     constexpr int COLS = VC * DA_WARPS, DP = 32 * JD, RW = 2 * DP + COLS, TB = 32 / VC;
     constexpr int PER = (CH * RW + 32 * DA_WARPS - 1) / (32 * DA_WARPS);
     static_assert(CH % TB == 0, "a chunk is whole batches of tokens");
     __shared__ __align__(16) float da_sm[2 * CH * RW];       // a token's row: q [DP], k [DP] (zeros behind D), the block's v [COLS]
+    __shared__ __align__(8) float da_coef[SSD ? 2 * CH * 2 : 2];       // SSD: a token's decay and dt
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int vb = blockIdx.x * COLS, v0 = vb + warp * VC, h = blockIdx.y, seg = blockIdx.z;
     const int start = seg_start[seg], len = seg_len[seg];
-    const float dec = decay[h];
-    float* st = state + (size_t)seg_slot[seg] * state_stride + (size_t)h * D * V;
+    const int g = SSD ? h / ssd.rep : h;                     // the head of the query and key rows
+    const float dec = SSD ? 0.f : decay[h], skip = SSD ? ssd.skip[h] : 0.f;
+    float* slot = state + (size_t)seg_slot[seg] * state_stride;
+    float* st = slot + (size_t)h * D * V;
+    auto at = [&](int d, int c) -> size_t { return SSD ? (size_t)(v0 + c) * D + d : (size_t)d * V + v0 + c; };
     xr_pdl_wait();
     float s[VC][JD];
+    // (SSD: a lane's JD elements of a column lie together: one access where they fall on a border of their size)
+    const bool whole = SSD && JD > 1 && D % JD == 0 && ((uintptr_t)st % (JD >= 4 ? 16 : 8)) == 0;
+    if (whole) {
 #pragma unroll
-    for (int j = 0; j < JD; j++) {
-        const int d = lane * JD + j;
+        for (int c = 0; c < VC; c++) {
+            const bool ok = lane * JD < D && v0 + c < V;
+            const float* p = st + at(lane * JD, ok ? c : 0);
+            if constexpr (JD % 4 == 0) {
 #pragma unroll
-        for (int c = 0; c < VC; c++) s[c][j] = (d < D && v0 + c < V) ? st[(size_t)d * V + v0 + c] : 0.f;
+                for (int j = 0; j < JD; j += 4) {
+                    const float4 x = ok ? *reinterpret_cast<const float4*>(p + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    s[c][j] = x.x; s[c][j + 1] = x.y; s[c][j + 2] = x.z; s[c][j + 3] = x.w;
+                }
+            } else if constexpr (JD == 2) {
+                const float2 x = ok ? *reinterpret_cast<const float2*>(p) : make_float2(0.f, 0.f);
+                s[c][0] = x.x; s[c][1] = x.y;
+            }
+        }
+    } else {
+#pragma unroll
+        for (int j = 0; j < JD; j++) {
+            const int d = lane * JD + j;
+#pragma unroll
+            for (int c = 0; c < VC; c++) s[c][j] = (d < D && v0 + c < V) ? st[at(d, c)] : 0.f;
+        }
     }
+    float coef_stage = 0.f;
     constexpr int PER4 = (CH * RW / 4 + 32 * DA_WARPS - 1) / (32 * DA_WARPS);
     float stage[VEC ? 1 : PER];
     float4 stage4[VEC ? PER4 : 1];
     // (loads that stay where they are written: left alone, the compiler moves them down to their use behind the walk to save
     // registers, and the chunk then waits for them one after the other)
     auto load = [&](int chunk) {
+        if (SSD && threadIdx.x < 2 * CH) {
+            const int i = chunk * CH + threadIdx.x / 2;
+            coef_stage = i < len ? xr_ld_now(ssd.coef + ((size_t)(start + i) * H + h) * 2 + (threadIdx.x & 1)) : 0.f;
+        }
         if constexpr (VEC) {
 #pragma unroll
             for (int k = 0; k < PER4; k++) {
@@ -351,8 +398,8 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
                 float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
                 if (tok < CH && i < len) {
                     const float* row = proj + (size_t)(start + i) * ldp;
-                    if (cc < DP) { if (cc < D) v = xr_ld_now4(reinterpret_cast<const float4*>(row + q_col + h * D + cc)); }
-                    else if (cc < 2 * DP) { if (cc - DP < D) v = xr_ld_now4(reinterpret_cast<const float4*>(row + k_col + h * D + cc - DP)); }
+                    if (cc < DP) { if (cc < D) v = xr_ld_now4(reinterpret_cast<const float4*>(row + q_col + g * D + cc)); }
+                    else if (cc < 2 * DP) { if (cc - DP < D) v = xr_ld_now4(reinterpret_cast<const float4*>(row + k_col + g * D + cc - DP)); }
                     else if (vb + cc - 2 * DP < V) v = xr_ld_now4(reinterpret_cast<const float4*>(row + v_col + h * V + vb + cc - 2 * DP));
                 }
                 stage4[k] = v;
@@ -367,8 +414,8 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
                 float v = 0.f;
                 if (tok < CH && i < len) {
                     const float* row = proj + (size_t)(start + i) * ldp;
-                    if (cc < DP) { if (cc < D) v = xr_ld_now(row + q_col + h * D + cc); }
-                    else if (cc < 2 * DP) { if (cc - DP < D) v = xr_ld_now(row + k_col + h * D + cc - DP); }
+                    if (cc < DP) { if (cc < D) v = xr_ld_now(row + q_col + g * D + cc); }
+                    else if (cc < 2 * DP) { if (cc - DP < D) v = xr_ld_now(row + k_col + g * D + cc - DP); }
                     else if (vb + cc - 2 * DP < V) v = xr_ld_now(row + v_col + h * V + vb + cc - 2 * DP);
                 }
                 stage[k] = v;
@@ -378,6 +425,7 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
         }
     };
     auto store = [&](int buf) {
+        if (SSD && threadIdx.x < 2 * CH) da_coef[buf * 2 * CH + threadIdx.x] = coef_stage;
         if constexpr (VEC) {
 #pragma unroll
             for (int k = 0; k < PER4; k++) {
@@ -411,6 +459,7 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
                 if (t0 + tb < here) {
                     const float* row = base + (t0 + tb) * RW;
                     float q[JD], k[JD], v[VC];
+                    float a = dec;
                     if constexpr (JD % 4 == 0) {
 #pragma unroll
                         for (int j = 0; j < JD; j += 4) {
@@ -437,11 +486,17 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
 #pragma unroll
                         for (int c = 0; c < VC; c++) v[c] = row[2 * DP + warp * VC + c];
                     }
+                    if constexpr (SSD) {
+                        const float2 ad = *reinterpret_cast<const float2*>(da_coef + ((ch & 1) * CH + t0 + tb) * 2);
+                        a = ad.x;
+#pragma unroll
+                        for (int c = 0; c < VC; c++) v[c] *= ad.y;
+                    }
 #pragma unroll
                     for (int j = 0; j < JD; j++) {
 #pragma unroll
                         for (int c = 0; c < VC; c++) {
-                            s[c][j] = fmaf(dec, s[c][j], k[j] * v[c]);
+                            s[c][j] = fmaf(a, s[c][j], k[j] * v[c]);
                             acc[tb * VC + c] = fmaf(s[c][j], q[j], acc[tb * VC + c]);
                         }
                     }
@@ -461,18 +516,40 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
             // read from its highest bit down is the sum's index
             const int mine = ((lane & 16) ? 16 : 0) + ((lane & 8) ? 8 : 0) + ((lane & 4) ? 4 : 0) + ((lane & 2) ? 2 : 0) + (lane & 1);
             const int tb = mine / VC, c = mine % VC;
-            if (t0 + tb < here && v0 + c < V) o[(size_t)(start + ch * CH + t0 + tb) * H * V + (size_t)h * V + v0 + c] = acc[0];
+            if (t0 + tb < here && v0 + c < V) {
+                float y = acc[0];
+                if constexpr (SSD) y = fmaf(skip, base[(t0 + tb) * RW + 2 * DP + warp * VC + c], y);
+                o[(size_t)(start + ch * CH + t0 + tb) * H * V + (size_t)h * V + v0 + c] = y;
+            }
         }
         if (ch + 1 < chunks) store((ch + 1) & 1);
         __syncthreads();
     }
+    if (whole) {
 #pragma unroll
-    for (int j = 0; j < JD; j++) {
-        const int d = lane * JD + j;
+        for (int c = 0; c < VC; c++) {
+            if (lane * JD >= D || v0 + c >= V) continue;
+            float* p = st + at(lane * JD, c);
+            if constexpr (JD % 4 == 0) {
 #pragma unroll
-        for (int c = 0; c < VC; c++)
-            if (d < D && v0 + c < V) st[(size_t)d * V + v0 + c] = s[c][j];
+                for (int j = 0; j < JD; j += 4) *reinterpret_cast<float4*>(p + j) = make_float4(s[c][j], s[c][j + 1], s[c][j + 2], s[c][j + 3]);
+            } else if constexpr (JD == 2) {
+                *reinterpret_cast<float2*>(p) = make_float2(s[c][0], s[c][1]);
+            }
+        }
+    } else {
+#pragma unroll
+        for (int j = 0; j < JD; j++) {
+            const int d = lane * JD + j;
+#pragma unroll
+            for (int c = 0; c < VC; c++)
+                if (d < D && v0 + c < V) st[at(d, c)] = s[c][j];
+        }
     }
+    if constexpr (SSD)
+        if (ssd.taps > 1)
+            xr_tail_update<float>(ssd.raw, ssd.ld_raw, slot + (size_t)H * V * D, start, len, ssd.CH, ssd.taps,
+                                  blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
 }
 
 // proj [n][ldp] float32: pre-activations of q at q_col [H][D], k at k_col [H][D], v at v_col [H][V] (`cols` columns from the first
@@ -495,11 +572,11 @@ XR_EXPORT int xr_decay_attention(float* proj, long long ldp, int q_col, int k_co
     // 16 bytes a load where every row, column offset and size falls on a 16-byte border
     const bool vec = !((D | V | ldp | q_col | k_col | v_col) & 3) && !((uintptr_t)proj & 15);
 #define DS_ARGS(JD, VC, CH) dim3((V + VC * DA_WARPS - 1) / (VC * DA_WARPS), H, n_seg), dim3(32 * DA_WARPS), 0, stream,                      \
-                            (const float*)proj, ldp, q_col, k_col, v_col, decay, state, state_stride, seg_start, seg_len, seg_slot, o, H, D, V, many ? 1 : 0
+                            (const float*)proj, ldp, q_col, k_col, v_col, decay, state, state_stride, seg_start, seg_len, seg_slot, o, H, D, V, many ? 1 : 0, SsdArgs{}
 #define DS1(JD, VC, CH, VEC)                                                                                                                 \
     do {                                                                                                                                     \
-        if (walk) xr_launch_behind((k_decay_scan<JD, VC, CH, VEC>), DS_ARGS(JD, VC, CH));                                                    \
-        else xr_launch((k_decay_scan<JD, VC, CH, VEC>), DS_ARGS(JD, VC, CH));                                                                \
+        if (walk) xr_launch_behind((k_decay_scan<JD, VC, CH, VEC, false>), DS_ARGS(JD, VC, CH));                                                    \
+        else xr_launch((k_decay_scan<JD, VC, CH, VEC, false>), DS_ARGS(JD, VC, CH));                                                                \
     } while (0)
 #define DS(JD, VC, CH)                                                                                                                       \
     do {                                                                                                                                     \
@@ -513,5 +590,106 @@ XR_EXPORT int xr_decay_attention(float* proj, long long ldp, int q_col, int k_co
 #undef DS
 #undef DS1
 #undef DS_ARGS
+    return xr_launch_status();
+}
+
+// ---------------------------------------------------------------------------------------------
+// (3): the convolution with its bias and silu, xbc [n][CH], and per token and head coef [n][H][2] = (exp(neg_a dt), dt), dt =
+// softplus(dt' + dt_bias).  A thread a column of xbc or a head's dt, TT tokens one after the other.  TAPS: taps known at
+// compile time (0: any number).
+// ---------------------------------------------------------------------------------------------
+template <int TAPS>
+__global__ void __launch_bounds__(256)
+k_ssd_prep(const float* __restrict__ proj, long long ldp, int x_col, int dt_col, const float* __restrict__ conv_w, const float* __restrict__ conv_b,
+           const float* __restrict__ dt_bias, const float* __restrict__ neg_a, const float* __restrict__ state, long long state_stride,
+           long long tail_off, const int* __restrict__ tok_seg, const int* __restrict__ seg_start, const int* __restrict__ seg_slot,
+           float* __restrict__ xbc, float* __restrict__ coef, int n, int CH, int H, int taps, int TT, int early) {
+    if (early) xr_pdl_launch();                  // (the walk behind it is a few long-lived blocks: see k_delta_prep)
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, t0 = blockIdx.y * TT, t1 = min(n, t0 + TT);
+    if (c >= CH + H) return;
+    if (c >= CH) {
+        const int h = c - CH;
+        const float bias = dt_bias[h], na = neg_a[h];
+        xr_pdl_wait();
+        for (int t = t0; t < t1; t++) {
+            const float z = proj[(size_t)t * ldp + dt_col + h] + bias;
+            const float dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+            *reinterpret_cast<float2*>(coef + ((size_t)t * H + h) * 2) = make_float2(expf(na * dt), dt);
+        }
+        return;
+    }
+    const int K = TAPS > 0 ? TAPS : taps;
+    const float* wc = conv_w + (size_t)c * K;
+    const float bias = conv_b[c];
+    float w[TAPS > 0 ? TAPS : 1];
+    if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) w[j] = wc[j];
+    }
+    xr_pdl_wait();
+    for (int t = t0; t < t1; t++) {
+        const int seg = tok_seg[t], i = t - seg_start[seg];
+        const float* x = proj + (size_t)t * ldp + x_col + c;
+        float acc = bias;
+        if (TAPS > 0 && i >= TAPS - 1) {                                   // every input is a row of this step
+            float v[TAPS > 0 ? TAPS : 1];
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) v[j] = x[-(long long)(TAPS - 1 - j) * ldp];
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) acc = fmaf(w[j], v[j], acc);
+        } else {
+            const float* tail = state + (size_t)seg_slot[seg] * state_stride + tail_off;
+            for (int j = K - 1; j >= 0; j--) {                             // oldest input first
+                const int ip = i - j;
+                const float v = ip >= 0 ? x[-(long long)j * ldp] : tail[(size_t)(K - 1 + ip) * CH + c];
+                acc = fmaf(wc[K - 1 - j], v, acc);
+            }
+        }
+        xbc[(size_t)t * CH + c] = rc_silu(acc);
+    }
+}
+
+// proj [n][ldp] float32: the convolution's inputs x [H][V], B [G][N], C [G][N] from x_col on, dt' [H] at dt_col.  conv_w [CH][taps]
+// (the last column the current token's), conv_b [CH], dt_bias, neg_a = -exp(A_log), skip [H]; all float32.
+// state [slots][state_stride] float32.  xbc [n][CH], coef [n][H][2] float32 scratch.  y [n][H V] float32: S^T C + D x.
+XR_EXPORT int xr_ssd(const float* proj, long long ldp, int x_col, int dt_col, const float* conv_w, const float* conv_b, const float* dt_bias,
+                     const float* neg_a, const float* skip, float* state, long long state_stride, const int* tok_seg, const int* seg_start,
+                     const int* seg_len, const int* seg_slot, float* xbc, float* coef, float* y, int n, int n_seg, int H, int G, int N, int V,
+                     int taps, cudaStream_t stream) {
+    if (n < 1 || n_seg < 1 || H < 1 || G < 1 || H % G || N < 1 || N > 256 || V < 1 || taps < 1 || taps > 64 || n_seg > 65535 || H > 65535)
+        return XR_ERR_ARG;
+    const int CH = H * V + 2 * G * N;
+    const long long tail_off = (long long)H * V * N;
+    if (state_stride < tail_off + (long long)(taps - 1) * CH) return XR_ERR_ARG;
+    const int TT = n > 64 ? 8 : 1, early = n <= 64 ? 1 : 0;
+    const dim3 gp((CH + H + 255) / 256, (n + TT - 1) / TT);
+    if (gp.y > 65535) return XR_ERR_ARG;
+#define SP(TAPS) xr_launch((k_ssd_prep<TAPS>), gp, dim3(256), 0, stream, proj, ldp, x_col, dt_col, conv_w, conv_b, dt_bias, neg_a, (const float*)state,      \
+                           state_stride, tail_off, tok_seg, seg_start, seg_slot, xbc, coef, n, CH, H, taps, TT, early)
+    if (taps == 4) SP(4);
+    else SP(0);
+#undef SP
+    const bool walk = n > 4 * n_seg;
+    const bool vec = !((N | V) & 3) && !((uintptr_t)xbc & 15);
+    const SsdArgs ssd{coef, skip, proj + x_col, ldp, CH, taps, H / G};
+#define SS_ARGS(VC) dim3((V + VC * DA_WARPS - 1) / (VC * DA_WARPS), H, n_seg), dim3(32 * DA_WARPS), 0, stream, (const float*)xbc, (long long)CH,            \
+                    H * V + G * N, H * V, 0, (const float*)nullptr, state, state_stride, seg_start, seg_len, seg_slot, y, H, N, V, 1, ssd
+#define SS1(JD, VC, CK, VEC)                                                                                                                 \
+    do {                                                                                                                                     \
+        if (walk) xr_launch_behind((k_decay_scan<JD, VC, CK, VEC, true>), SS_ARGS(VC));                                                      \
+        else xr_launch((k_decay_scan<JD, VC, CK, VEC, true>), SS_ARGS(VC));                                                                  \
+    } while (0)
+#define SS(JD, VC, CK)                                                                                                                       \
+    do {                                                                                                                                     \
+        if (vec) SS1(JD, VC, CK, true);                                                                                                      \
+        else SS1(JD, VC, CK, false);                                                                                                         \
+    } while (0)
+    if (N <= 32) SS(1, 2, 16);
+    else if (N <= 64) SS(2, 2, 16);
+    else if (N <= 128) SS(4, 2, 16);
+    else SS(8, 4, 8);
+#undef SS
+#undef SS1
+#undef SS_ARGS
     return xr_launch_status();
 }

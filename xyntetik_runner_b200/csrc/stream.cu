@@ -201,6 +201,56 @@ XR_EXPORT int xr_row_norm_gate(const float* o, const float* g, long long ld_g, c
     return xr_launch_status();
 }
 
+// ---------------------------------------------------------------------------
+// A gate AHEAD of a norm over groups of columns: v = o[t][i] * silu(g[t][i]); y[t][i] = v / sqrt(mean of v^2 over the column's group + eps)
+// * w[i].  o, g float32 (rows of g ld_g apart), y in the activation dtype; `groups` equal groups.  A block per (row, group); its
+// first SGN_KEEP values a thread stay in registers between the two passes, further ones are computed again.
+// ---------------------------------------------------------------------------
+#define SGN_KEEP 16
+
+__device__ __forceinline__ float st_silu_gated(float o, float g) { return o * (g < -80.0f ? 0.0f : g / (1.0f + expf(-g))); }
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+k_silu_gate_norm(const float* __restrict__ o, const float* __restrict__ g, long long ld_g, const float* __restrict__ w, T* __restrict__ y,
+                 int width, int per, float eps) {
+    xr_pdl_launch();
+    __shared__ float scratch[33];
+    xr_pdl_wait();
+    const int c0 = blockIdx.y * per;
+    const float* src = o + (size_t)blockIdx.x * width + c0;
+    const float* gate = g + (size_t)blockIdx.x * ld_g + c0;
+    float v[SGN_KEEP], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < SGN_KEEP; k++) {
+        const int i = threadIdx.x + k * blockDim.x;
+        v[k] = i < per ? st_silu_gated(src[i], gate[i]) : 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < SGN_KEEP; k++) ss = fmaf(v[k], v[k], ss);
+    for (int i = threadIdx.x + SGN_KEEP * blockDim.x; i < per; i += blockDim.x) { const float x = st_silu_gated(src[i], gate[i]); ss = fmaf(x, x, ss); }
+    ss = xr_block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)per + eps);
+    T* out = y + (size_t)blockIdx.x * width + c0;
+#pragma unroll
+    for (int k = 0; k < SGN_KEEP; k++) {
+        const int i = threadIdx.x + k * blockDim.x;
+        if (i < per) out[i] = xr_from_f32<T>(v[k] * inv * w[c0 + i]);
+    }
+    for (int i = threadIdx.x + SGN_KEEP * blockDim.x; i < per; i += blockDim.x) out[i] = xr_from_f32<T>(st_silu_gated(src[i], gate[i]) * inv * w[c0 + i]);
+}
+
+XR_EXPORT int xr_silu_gate_norm(const float* o, const float* g, long long ld_g, const float* w, void* y, int dtype, int n, int width, int groups,
+                                float eps, cudaStream_t stream) {
+    if (n < 1 || width < 1 || groups < 1 || width % groups || groups > 65535) return XR_ERR_ARG;
+    const int per = width / groups, threads = per >= 256 ? 256 : (per + 31) / 32 * 32;
+    const dim3 grid(n, groups);
+    if (dtype == XR_F32) xr_launch((k_silu_gate_norm<float>), grid, dim3(threads), 0, stream, o, g, ld_g, w, (float*)y, width, per, eps);
+    else if (dtype == XR_BF16) xr_launch((k_silu_gate_norm<__nv_bfloat16>), grid, dim3(threads), 0, stream, o, g, ld_g, w, (__nv_bfloat16*)y, width, per, eps);
+    else return XR_ERR_ARG;
+    return xr_launch_status();
+}
+
 // out[i] = x[i] in the activation dtype
 template <typename T>
 __global__ void k_cast_rows(const float* __restrict__ x, T* __restrict__ out, size_t total) {

@@ -110,7 +110,7 @@ class LoadedModel:
         self.groups: List[CacheGroupLayout] = []
         self.layers: List[LayerRuntime] = []
         self.state_needs: List[Tuple[int, StateNeed]] = []
-        keys: Dict[Tuple[int, int, Optional[int], int], int] = {}
+        keys: Dict[Tuple[int, int, Optional[int], int, int], int] = {}
         for i, e in enumerate(plan.schedule):
             mixer = plan.blocks[e.layer].mixer
             lay = LayerRuntime(entry=i)
@@ -120,11 +120,11 @@ class LoadedModel:
                     src = self.layers[e.cache_from]
                     lay.group, lay.layer_in_group, lay.writes_cache = src.group, src.layer_in_group, False
                 else:
-                    key = (need.kv_heads, need.head_dim, need.window, need.planes)
+                    key = (need.kv_heads, need.head_dim, need.window, need.planes, need.keep_first)
                     if key not in keys:
                         keys[key] = len(self.groups)
-                        name = "full" if need.window is None else f"window{need.window}"
-                        self.groups.append(CacheGroupLayout(GroupSpec(f"{name}:{need.planes}x{need.kv_heads}x{need.head_dim}", need.window),
+                        name = "full" if need.window is None else f"window{need.window}" + (f"+{need.keep_first}" if need.keep_first else "")
+                        self.groups.append(CacheGroupLayout(GroupSpec(f"{name}:{need.planes}x{need.kv_heads}x{need.head_dim}", need.window, need.keep_first),
                                                             need.kv_heads, need.head_dim, planes=need.planes))
                     g = keys[key]
                     lay.group, lay.layer_in_group, lay.writes_cache = g, self.groups[g].n_layers, True

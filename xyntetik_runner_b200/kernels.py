@@ -53,18 +53,18 @@ def _declare(L: ctypes.CDLL) -> None:
         "xr_act_mul": [_vp, _vp, _i, _i, _i, _i, _i, _f, _vp],
         "xr_residual_add": [_vp, _vp, _i, _i, _i, _vp],
         "xr_gemm_simt": [_vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _ll, _ll, _vp],
-        "xr_attention_simt": [_vp, _vp, _i, _vp, _vp, _vp, _vp, _ll, _ll, _ll, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _f, _vp],
+        "xr_attention_simt": [_vp, _vp, _i, _vp, _vp, _vp, _vp, _ll, _ll, _ll, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _f, _i, _vp, _i, _vp],
         "xr_gemm_tc": [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _i, _ll, _ll, _vp, _ll, _vp, _i, _i, ctypes.POINTER(ctypes.c_int), _i, _vp],
         "xr_finish_add_rmsnorm": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _vp],
         "xr_finish_plain": [_vp, _i, _vp, _vp, _i, _i, _i, _i, _ll, _vp],
         "xr_finish_rope_store": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
         "xr_attention_mma": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _ll, _ll, _i, _i, _i, _i, _i, _i, _i, _f,
-                             _i, _i, _i, _i, _i, _vp, _ll, _i, _i, _vp, _vp, _i, _i, _ll, _vp, _f, _vp],
+                             _i, _i, _i, _i, _i, _vp, _ll, _i, _i, _vp, _vp, _i, _i, _ll, _vp, _f, _i, _vp, _i, _vp],
         "xr_attention_mma_splits": [_i, _i, _ll],
         "xr_attention_even_launches": [],
         "xr_attention_wait_probe": [_vp, _vp, ctypes.c_uint, _vp],
         "xr_attention_tc_supported": [_i, _i, _i, _i],
-        "xr_attention_tc": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _ll, _ll, _i, _i, _vp, _f, _vp],
+        "xr_attention_tc": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _ll, _ll, _i, _i, _vp, _f, _i, _vp, _i, _vp],
         "xr_sample": [_vp, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp],
         "xr_sample_one_block": [_vp, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp],
         "xr_logprob": [_vp, _ll, _i, _i, _vp, _vp, _vp],
@@ -82,7 +82,7 @@ def _declare(L: ctypes.CDLL) -> None:
         "xr_heads_gather": [_vp, _ll, _i, _vp, _i, _i, _i, _i, _vp],
         "xr_heads_scatter_gate": [_vp, _vp, _vp, _ll, _i, _i, _i, _i, _i, _vp],
         "xr_qk_norm_rope_store": [_vp, _i, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i,
-                                  _vp, _i, _vp, _i, _f, _i, _vp],
+                                  _vp, _i, _vp, _i, _f, _i, _vp, _i, _f, _vp],
         "xr_rmsnorm_act": [_vp, _i, _ll, _vp, _vp, _ll, _i, _i, _f, _vp],
         "xr_delta": [_vp, _i, _ll, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
         "xr_head_norm_gate": [_vp, _vp, _i, _ll, _vp, _i, _i, _vp, _i, _i, _i, _i, _f, _vp],
@@ -93,7 +93,8 @@ def _declare(L: ctypes.CDLL) -> None:
         "xr_gemm_tc_grouped": [_vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _i, _ll, _ll, _i, _vp, _i, _vp, _vp],
         "xr_moe_tile_rows": [],
         "xr_moe_gemm": [_vp, _i, _ll, _vp, _i, _vp, _i, _ll, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _vp],
-        "xr_moe_combine": [_vp, _vp, _vp, _vp, _i, _i, _i, _vp],
+        "xr_route_groups": [_vp, _vp, _vp, _i, _i, _i, _vp, _i, _i, _f, _vp],
+        "xr_moe_combine": [_vp, _vp, _vp, _vp, _vp, _i, _ll, _i, _i, _i, _vp],
         "xr_embed_pair": [_vp, _vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _ll, _vp],
         "xr_last_token": [_vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _vp],
         "xr_norm_add": [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp, _vp, _i, _vp],
@@ -103,6 +104,8 @@ def _declare(L: ctypes.CDLL) -> None:
         "xr_rglru": [_vp, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
                      _f, _vp],
         "xr_row_norm_gate": [_vp, _vp, _ll, _vp, _vp, _i, _i, _i, _f, _f, _vp],
+        "xr_ssd": [_vp, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
+        "xr_silu_gate_norm": [_vp, _vp, _ll, _vp, _vp, _i, _i, _i, _i, _f, _vp],
         "xr_decay_attention": [_vp, _ll, _i, _i, _i, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     }
     for name, args in sig.items():
@@ -206,10 +209,10 @@ def rope_store(qkv: torch.Tensor, positions, tok_seg, block_tables, inv_freq: Op
     _count()
 
 
-ACT_NONE, ACT_SILU, ACT_GELU_TANH, ACT_SWISH_CLAMP = 0, 1, 2, 3
+ACT_NONE, ACT_SILU, ACT_GELU_TANH, ACT_SWISH_CLAMP, ACT_RELU2 = 0, 1, 2, 3, 4
 # "swish_clamp" exists for gated products only and takes a `limit`: with g' = min(g, limit) and u' = u clamped to
-# [-limit, limit] the product stores g' sigmoid(1.702 g') (u' + 1).
-ACTIVATIONS = {"none": ACT_NONE, "silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH, "swish_clamp": ACT_SWISH_CLAMP}
+# [-limit, limit] the product stores g' sigmoid(1.702 g') (u' + 1).  "relu2" is the square of relu.
+ACTIVATIONS = {"none": ACT_NONE, "silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH, "swish_clamp": ACT_SWISH_CLAMP, "relu2": ACT_RELU2}
 
 
 def rmsnorm_act(inp: torch.Tensor, w: torch.Tensor, out: torch.Tensor, eps: float) -> None:
@@ -227,7 +230,8 @@ def qk_norm_rope_store(inp: torch.Tensor, q_out: torch.Tensor, positions, tok_se
                        q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor], cache_k_ptr: Optional[int], page_stride: int, v_offset: int,
                        H: int, K: int, D: int, Vd: int, hd: int, rotary_dim: int, max_pages: int, page_size: int, adjacent: bool,
                        eps: float, unit_norm: bool = False, q_coef: float = 0.0, q_every: int = 0, partial: Optional[torch.Tensor] = None,
-                       splits: int = 0, bias: Optional[torch.Tensor] = None, mscale: float = 1.0, norm_after: bool = False) -> None:
+                       splits: int = 0, bias: Optional[torch.Tensor] = None, mscale: float = 1.0, norm_after: bool = False,
+                       v_first: Optional[torch.Tensor] = None, v_lambda: Optional[float] = None) -> None:
     """inp [n, >= (H + K) D + K Vd] (rows may be strided): Q heads, K heads (D each), V heads (Vd each).  Every Q and K head is
     RMS-normed with the weight q_w / k_w (float32 [D], shared by the heads; None: no norm), its first `rotary_dim` elements rotated
     (freq: float64 [rotary_dim / 2]); Q goes to q_out [n, *] (head h at column h * hd), K and V into the token's cache rows, every
@@ -235,8 +239,12 @@ def qk_norm_rope_store(inp: torch.Tensor, q_out: torch.Tensor, positions, tok_se
     and K head is divided by its root mean square all the same.  `q_every` > 0: the Q heads of the token at position p are
     multiplied by 1 + q_coef ln(floor((p + 1) / q_every) + 1).  `partial` (float32 [splits][n][inp.shape[1]], with `bias`): the rows are
     still the partial sums of a product cut along K; the kernel sums them (+ bias) into `inp`, every column, before it reads them.
-    `mscale` multiplies every cosine and sine; `norm_after` (with `unit_norm`): the root mean square is that of the rotated head."""
-    _dev(positions, tok_seg, block_tables, freq, q_w, k_w, partial, bias)
+    `mscale` multiplies every cosine and sine; `norm_after` (with `unit_norm`): the root mean square is that of the rotated head.
+    `v_first` [n, K Vd] (inp's dtype): with `v_lambda` None the values are also left there; with a number what is cached is
+    (1 - v_lambda) v + v_lambda v_first."""
+    _dev(positions, tok_seg, block_tables, freq, q_w, k_w, partial, bias, v_first)
+    assert v_first is None or (v_first.shape == (inp.shape[0], K * Vd) and v_first.dtype == inp.dtype)
+    assert v_lambda is None or v_first is not None
     n = inp.shape[0]
     assert partial is None or (partial.dtype == torch.float32 and splits >= 1 and partial.numel() >= splits * n * inp.shape[1])
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == inp.shape[1])
@@ -248,6 +256,7 @@ def qk_norm_rope_store(inp: torch.Tensor, q_out: torch.Tensor, positions, tok_se
                                        cache_k_ptr, page_stride, v_offset, n, H, K, D, Vd, hd, rotary_dim, max_pages, page_size,
                                        int(adjacent), float(eps), int(unit_norm), float(q_coef), int(q_every), _ptr(partial), int(splits),
                                        _ptr(bias) if partial is not None else None, inp.shape[1], float(mscale), int(norm_after),
+                                       _ptr(v_first), 0 if v_first is None else (1 if v_lambda is None else 2), float(v_lambda or 0.0),
                                        _stream()),
            "qk_norm_rope_store")
     _count()
@@ -292,20 +301,32 @@ def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optiona
     _count()
 
 
+def _check_bias(bias: Optional[torch.Tensor], H: int) -> None:
+    _dev(bias)
+    assert bias is None or (bias.dtype == torch.float32 and bias.dim() == 2 and bias.shape[0] == H and bias.shape[1] >= 1)
+
+
+def _bias_len(bias: Optional[torch.Tensor]) -> int:
+    return 0 if bias is None else bias.shape[1]
+
+
 def attention_simt(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, cache_k_ptr: int, positions, tok_seg,
                    block_tables, page_stride: int, v_offset: int, H: int, K: int, hd: int, max_pages: int,
-                   page_size: int, window: int, scale: float, sink: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
+                   page_size: int, window: int, scale: float, sink: Optional[torch.Tensor] = None, softcap: float = 0.0,
+                   keep_first: int = 0, bias: Optional[torch.Tensor] = None) -> None:
     """Causal attention of every token of the step over its request's pages, float32 arithmetic.  `sink`: float32 [H];
     exp(sink[h]) joins the denominator of head h's softmax once (it has no key and no value).  `softcap` c > 0: every scaled
-    score s becomes c tanh(s / c)."""
+    score s becomes c tanh(s / c).  `keep_first`: with a window, a request's first keys stay visible behind it.  `bias`
+    (float32 [H, L]): the query of head h at distance d from a key adds scale * bias[h, min(d, L - 1)] to the score."""
     _dev(out, positions, tok_seg, block_tables, sink)
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == H)
     n = out.shape[0]
+    _check_bias(bias, H)
     assert out.shape[1] == H * hd and q.dtype == out.dtype
     _check(lib().xr_attention_simt(q.data_ptr(), out.data_ptr(), dtype_code(out.dtype), cache_k_ptr,
                                    positions.data_ptr(), tok_seg.data_ptr(), block_tables.data_ptr(), page_stride,
                                    v_offset, q_row_stride, n, H, K, hd, max_pages, page_size, window, float(scale),
-                                   _ptr(sink), float(softcap), _stream()), "attention_simt")
+                                   _ptr(sink), float(softcap), int(keep_first), _ptr(bias), _bias_len(bias), _stream()), "attention_simt")
     _count()
 
 
@@ -632,7 +653,8 @@ def attention_mma(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, cache_k
                   v_offset: int, H: int, K: int, hd: int, max_pages: int, page_size: int, window: int, scale: float,
                   n_seg: int, max_seg_len: int, max_kv_len: int, splits: int, any_short: bool, any_long: bool,
                   group: Optional[tuple] = None, uneven: bool = False, row_tiles: int = 0,
-                  sink: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
+                  sink: Optional[torch.Tensor] = None, softcap: float = 0.0, keep_first: int = 0,
+                  bias: Optional[torch.Tensor] = None) -> None:
     """Causal attention over the pages on tensor cores (bfloat16); `softcap` c > 0: every scaled score s becomes c tanh(s / c).  Portions with at most 16 packed rows
     (tokens x heads per kv head) go through the key-split kernel and need `part_acc` [n_seg*K*splits*16*hd]
     and `part_ml` [n_seg*K*splits*32] float32 scratch; longer portions through the row-tiled kernel.
@@ -641,8 +663,9 @@ def attention_mma(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, cache_k
     `uneven`: the requests' lengths differ much; the kernel then cuts the tiles of all requests into even shares from
     fewer requests on than it does otherwise.  row_tiles: ``long_row_tiles(lengths, H // K, 64)``, which sizes the
     row-tiled kernel's grid exactly; 0: every portion gets the blocks of the longest.  `sink`: float32 [H]; exp(sink[h])
-    joins the denominator of head h's softmax once."""
+    joins the denominator of head h's softmax once.  `keep_first`, `bias`: see ``attention_simt`` (a bias goes without a cap)."""
     _dev(out, seg_start, seg_len, seg_pos0, block_tables, part_acc, part_ml, sink)
+    _check_bias(bias, H)
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == H)
     assert q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and out.shape[1] == H * hd
     if any_short:
@@ -656,7 +679,7 @@ def attention_mma(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, cache_k
                                   group[0] if group else None, group[1] if group else 0, group[2] if group else 1,
                                   group[3] if group else 0, ws.status.data_ptr() if group else None,
                                   ws.flags.data_ptr() if group else None, ws.flags.numel() if group else 0, int(uneven),
-                                  row_tiles, _ptr(sink), float(softcap), _stream()), "attention_mma")
+                                  row_tiles, _ptr(sink), float(softcap), int(keep_first), _ptr(bias), _bias_len(bias), _stream()), "attention_mma")
     _count((1 if any_long else 0) + (2 if any_short else 0))
 
 
@@ -666,11 +689,14 @@ def attention_tc_supported(dtype: torch.dtype, H: int, K: int, hd: int, page_siz
 
 def attention_tc(qkv: torch.Tensor, out: torch.Tensor, seg_start, seg_len, seg_pos0, block_tables, group: tuple,
                  H: int, K: int, hd: int, max_pages: int, page_size: int, window: int, scale: float, n_seg: int,
-                 max_seg_len: int, row_tiles: int = 0, sink: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
+                 max_seg_len: int, row_tiles: int = 0, sink: Optional[torch.Tensor] = None, softcap: float = 0.0,
+                 keep_first: int = 0, bias: Optional[torch.Tensor] = None) -> None:
     """Causal attention of the portions with more than 16 packed rows on tcgen05 (S and O in tensor memory).
     qkv: the step's fused rows (Q heads first); group = (pointer to the cache group's array, pages, layers, layer).
     row_tiles: ``long_row_tiles(lengths, H // K, 128)``, which sizes the grid exactly; 0: every portion gets the blocks
-    of the longest.  `sink`: float32 [H]; exp(sink[h]) joins the denominator of head h's softmax once."""
+    of the longest.  `sink`: float32 [H]; exp(sink[h]) joins the denominator of head h's softmax once.  `keep_first`, `bias`:
+    see ``attention_simt`` (a bias goes without a cap)."""
+    _check_bias(bias, H)
     _dev(qkv, out, seg_start, seg_len, seg_pos0, block_tables, sink)
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == H)
     n = qkv.shape[0]
@@ -679,7 +705,7 @@ def attention_tc(qkv: torch.Tensor, out: torch.Tensor, seg_start, seg_len, seg_p
     _check(lib().xr_attention_tc(qkv.data_ptr(), out.data_ptr(), group[0], seg_start.data_ptr(), seg_len.data_ptr(),
                                  seg_pos0.data_ptr(), block_tables.data_ptr(), status.data_ptr(), qkv.stride(0), n, n_seg,
                                  H, K, hd, max_pages, page_size, window, float(scale), max_seg_len, row_tiles, group[1], group[2],
-                                 group[3], _ptr(sink), float(softcap), _stream()), "attention_tc")
+                                 group[3], _ptr(sink), float(softcap), int(keep_first), _ptr(bias), _bias_len(bias), _stream()), "attention_tc")
     _count()
 
 
@@ -938,6 +964,21 @@ def route_topk(z: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, top: int, 
     _count()
 
 
+def route_groups(z: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, top: int, correction: Optional[torch.Tensor] = None, groups: int = 1,
+                 keep: int = 1, scale: float = 1.0) -> None:
+    """The choice with scores s = softmax(z[t]) over all E outputs (identity experts included), by c = s + correction (float32 [E],
+    optional): of `groups` equal groups of neighbours the `keep` with the largest c stay, of their outputs the `top` largest c are
+    chosen (ties: the lower index), and the weights are scale * s, not renormalised."""
+    _dev(z, ids, wts, correction)
+    n, E = z.shape
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E)
+    assert z.dtype == torch.float32 and ids.dtype == torch.int32 and wts.dtype == torch.float32
+    assert ids.shape == (n, top) and wts.shape == (n, top)
+    _check(lib().xr_route_groups(z.data_ptr(), ids.data_ptr(), wts.data_ptr(), n, E, top, _ptr(correction), int(groups), int(keep), float(scale),
+                                 _stream()), "route_groups")
+    _count()
+
+
 def moe_tile_rows() -> int:
     """Rows per tile of the FMA kernel of the experts' products (the alignment its plan needs)."""
     return int(lib().xr_moe_tile_rows())
@@ -951,7 +992,7 @@ def moe_max_tiles(pairs: int, E: int, align: int) -> int:
 def moe_plan(ids: torch.Tensor, row_src, pair_row, tile_group, E: int, align: int) -> None:
     """Sort the (token, choice) pairs by expert on the device, every expert's rows starting at a multiple of `align`:
     row_src [max_tiles * align] (pair of a row, -1: padding), pair_row [pairs], tile_group [max_tiles] (expert of a
-    tile, -1: no rows); see k_moe_plan in csrc/moe.cu."""
+    tile, -1: no rows); see k_moe_plan in csrc/moe.cu.  An id of E or more has no row (pair_row -1)."""
     _dev(ids, row_src, pair_row, tile_group)
     pairs = ids.numel()
     max_tiles = moe_max_tiles(pairs, E, align)
@@ -1007,12 +1048,14 @@ def gemm_tc_grouped(x: torch.Tensor, w_packed: torch.Tensor, out: torch.Tensor, 
     _count()
 
 
-def moe_combine(d: torch.Tensor, z: torch.Tensor, wts: torch.Tensor, pair_row: torch.Tensor, top: int) -> None:
-    """d[t] += sum_j wts[t, j] * z[pair_row[t * top + j]] (float32)."""
+def moe_combine(d: torch.Tensor, z: torch.Tensor, wts: torch.Tensor, pair_row: torch.Tensor, top: int, h: Optional[torch.Tensor] = None) -> None:
+    """d[t] += sum_j wts[t, j] * z[pair_row[t * top + j]] (float32); a pair without a row (-1) adds wts[t, j] * h[t]."""
     _dev(d, z, wts, pair_row)
     n, width = d.shape
     assert d.dtype == torch.float32 and z.dtype == torch.float32 and z.shape[1] == width
-    _check(lib().xr_moe_combine(d.data_ptr(), z.data_ptr(), wts.data_ptr(), pair_row.data_ptr(), n, width, top, _stream()), "moe_combine")
+    assert h is None or (h.is_cuda and h.shape == d.shape and h.stride(1) == 1)
+    _check(lib().xr_moe_combine(d.data_ptr(), z.data_ptr(), wts.data_ptr(), pair_row.data_ptr(), _ptr(h), 0 if h is None else dtype_code(h.dtype),
+                                0 if h is None else h.stride(0), n, width, top, _stream()), "moe_combine")
     _count()
 
 
@@ -1140,3 +1183,39 @@ def decay_attention(proj: torch.Tensor, cols, decay: torch.Tensor, state: torch.
                                     state.stride(0), seg_start.data_ptr(), seg_len.data_ptr(), seg_slot.data_ptr(), o.data_ptr(), n, n_seg, H, D, V,
                                     _stream()), "decay_attention")
     _count(2 if n > 16 else 1)
+
+
+def ssd_state_floats(H: int, G: int, N: int, V: int, taps: int) -> int:
+    """float32 values per request slot: S [H][V][N], then the last taps - 1 inputs of the convolution's H V + 2 G N channels."""
+    return H * V * N + (taps - 1) * (H * V + 2 * G * N)
+
+
+def ssd(proj: torch.Tensor, x_col: int, dt_col: int, conv_w, conv_b, dt_bias, neg_a, skip, state: torch.Tensor, tok_seg, seg_start, seg_len, seg_slot,
+        xbc: torch.Tensor, coef: torch.Tensor, y: torch.Tensor, n_seg: int, H: int, G: int, N: int, V: int, taps: int) -> None:
+    """The state-space dual recurrence of Mamba-2 over the step's tokens, request by request, from and into `state`: S <- a S + dt B x^T,
+    y = S^T C + skip x, with a = exp(neg_a dt), dt = softplus(dt' + dt_bias).  proj float32 [n, *] (rows may be strided): the
+    convolution's inputs x [H V], B [G N], C [G N] at x_col, dt' [H] at dt_col.  xbc [n, H V + 2 G N] and coef [n, 2 H] float32
+    scratch; y float32 [n, H V].  See csrc/recurrent.cu."""
+    _dev(conv_w, conv_b, dt_bias, neg_a, skip, state, tok_seg, seg_start, seg_len, seg_slot, xbc, coef, y)
+    n, CH = proj.shape[0], H * V + 2 * G * N
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= max(x_col + CH, dt_col + H)
+    assert all(t.dtype == torch.float32 for t in (conv_w, conv_b, dt_bias, neg_a, skip, state, xbc, coef, y))
+    assert conv_w.shape == (CH, taps) and conv_b.numel() == CH and all(t.numel() == H for t in (dt_bias, neg_a, skip))
+    assert state.dim() == 2 and state.shape[1] >= ssd_state_floats(H, G, N, V, taps)
+    assert xbc.shape == (n, CH) and coef.numel() >= 2 * n * H and y.shape == (n, H * V)
+    _check(lib().xr_ssd(proj.data_ptr(), proj.stride(0), x_col, dt_col, conv_w.data_ptr(), conv_b.data_ptr(), dt_bias.data_ptr(), neg_a.data_ptr(),
+                        skip.data_ptr(), state.data_ptr(), state.stride(0), tok_seg.data_ptr(), seg_start.data_ptr(), seg_len.data_ptr(),
+                        seg_slot.data_ptr(), xbc.data_ptr(), coef.data_ptr(), y.data_ptr(), n, n_seg, H, G, N, V, taps, _stream()), "ssd")
+    _count(2)
+
+
+def silu_gate_norm(o: torch.Tensor, gate: torch.Tensor, gate_col: int, w: torch.Tensor, y: torch.Tensor, groups: int, eps: float) -> None:
+    """v = o * silu(gate[:, gate_col:gate_col + width]); y = v / sqrt(mean of v^2 over each of `groups` equal groups of columns + eps) * w:
+    the gate comes ahead of the norm.  o, gate (rows may be strided), w float32, y in the activation dtype."""
+    _dev(o, w, y)
+    n, width = o.shape
+    assert o.dtype == torch.float32 and gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[1] >= gate_col + width
+    assert w.dtype == torch.float32 and w.numel() == width and y.shape == (n, width)
+    _check(lib().xr_silu_gate_norm(o.data_ptr(), gate.data_ptr() + 4 * gate_col, gate.stride(0), w.data_ptr(), y.data_ptr(), dtype_code(y.dtype),
+                                   n, width, int(groups), float(eps), _stream()), "silu_gate_norm")
+    _count()

@@ -9,10 +9,11 @@ from .embedding import Embedding, Head, PairEmbedding
 from .feed_forward import GatedFeedForward, MLP, SwiGLU
 from .latent_attention import LatentAttention
 from .linear import Linear
+from .mamba2 import Mamba2
 from .mlstm import MLSTM
 from .moe import RoutedExperts
 from .norm import RMSNorm, ScalarRMSNorm
-from .position import NoPosition, Rope, YarnRope
+from .position import DistanceBuckets, NoPosition, Rope, YarnRope
 from .rglru import GatedLinearRecurrence
 from .side_by_side import SideBySide
 from .stream import DepthAverage, StreamJoin, StreamStep

@@ -29,6 +29,11 @@ value of position j is turned by j over all its Vd elements (pair m by j base^(-
 at position i is turned back by -i, so that what a query reads of a value depends on their distance.  `softcap` c: every scaled
 score s becomes c tanh(s / c).  `sink=0.0` (a number instead of a tensor's name): a sink of that logit for every head, which adds
 exp(sink) to every softmax's denominator.  `out_scale` multiplies the heads' outputs before the output product.
+
+`keep_first` n (with a window): a request's first n keys stay visible behind the window, in their own positions; the pages that
+hold them stay held.  `distance_bias=(name, far)`: a learned table [rows, H] by distance joins the scaled scores, row
+``DistanceBuckets(rows, far)`` of the distance from query to key.  `value_share` lets layers share values: "first" leaves the
+layer's values of the step's tokens for the layers behind it, "mix" caches (1 - l) v + l v_first, l the number in the tensor `v_mix`.
 """
 from __future__ import annotations
 
@@ -43,6 +48,7 @@ from .. import kernels
 from ..weights.loader import TensorSpec
 from .base import KVNeed, Mixer, PositionEncoding, register_mixer
 from .linear import Linear
+from .position import DistanceBuckets
 
 # Which attention kernels the mixer may use (module attributes, so that a test can compare paths): the mma.sync kernels
 # for bfloat16 (else the float32-arithmetic kernel), the tcgen05 kernel for prompt portions, bulk copies in the decode
@@ -63,7 +69,8 @@ class GQAAttention(Mixer):
                  q_norm: str = "q.norm", k_norm: str = "k.norm", bias_suffix: str = ".bias", out_bias: Optional[bool] = None,
                  q_temp: Optional[tuple] = None, sink=None, gate: Optional[str] = None, g: str = "g",
                  norm_after_rotation: bool = False, value_rotation: Optional[tuple] = None, softcap: Optional[float] = None,
-                 out_scale: float = 1.0):
+                 out_scale: float = 1.0, keep_first: int = 0, distance_bias: Optional[tuple] = None,
+                 value_share: Optional[str] = None, v_mix: str = "vmix"):
         if heads % kv_heads:
             raise ValueError("heads must be a multiple of kv_heads")
         if qk_norm not in (False, True, "unit"):
@@ -76,10 +83,19 @@ class GQAAttention(Mixer):
             raise ValueError(f"{prefix}: norm_after_rotation goes with qk_norm='unit'")
         if value_rotation is not None and (len(value_rotation) != 2 or value_rotation[1] not in ("half", "adjacent")):
             raise ValueError(f"{prefix}: value_rotation is (base, 'half' or 'adjacent')")
+        if value_share not in (None, "first", "mix"):
+            raise ValueError(f"{prefix}: value_share is None, 'first' or 'mix'")
+        if value_share is not None and value_rotation is not None:
+            raise ValueError(f"{prefix}: shared values are not rotated")
+        if distance_bias is not None and (len(distance_bias) != 2 or softcap):
+            raise ValueError(f"{prefix}: distance_bias is (tensor name, distance of the last bucket) and goes without a cap on the scores")
+        if keep_first < 0:
+            raise ValueError(f"{prefix}: keep_first {keep_first}")
         self.D = head_dim                                      # query/key elements per head
         self.Vd = head_dim if value_dim is None else value_dim  # value elements per head
         # the general path: a norm per head, or values of another size than keys
-        self.general = bool(qk_norm) or self.Vd != self.D or q_temp is not None or gate is not None or value_rotation is not None
+        self.general = bool(qk_norm) or self.Vd != self.D or q_temp is not None or gate is not None or \
+            value_rotation is not None or value_share is not None
         # head size of the cache and of the attention kernels
         hd = -(-max(self.D, self.Vd) // 16) * 16 if self.general else head_dim
         if not (1 <= hd <= 256):
@@ -98,6 +114,11 @@ class GQAAttention(Mixer):
         self.norm_after, self.value_rotation = bool(norm_after_rotation), value_rotation
         self.softcap = float(softcap) if softcap else 0.0
         self.out_scale = float(out_scale)
+        self.keep_first = int(keep_first) if window is not None else 0
+        self.bias_name, self.bias_far = (None, 0.0) if distance_bias is None else (prefix + distance_bias[0], float(distance_bias[1]))
+        if distance_bias is not None and not self.scale > 0:
+            raise ValueError(f"{prefix}: a distance bias needs a positive score scale")
+        self.value_share, self.v_mix_name, self.v_lambda, self.dist_bias = value_share, prefix + v_mix, None, None
         if value_rotation is not None and self.Vd % 2:
             raise ValueError(f"{prefix}: rotated values need an even value size")
         self.vfreq64 = None
@@ -109,7 +130,7 @@ class GQAAttention(Mixer):
         self.q_norm_w = self.k_norm_w = self.freq64 = None
 
     def kv_need(self):
-        return KVNeed(self.K, self.hd, self.window)
+        return KVNeed(self.K, self.hd, self.window, keep_first=self.keep_first)
 
     def tensors(self):
         q, k, v, o = (self.prefix + n for n in self.proj)
@@ -129,6 +150,11 @@ class GQAAttention(Mixer):
             t[self.gate_name + sfx] = TensorSpec((self.gate_cols, self.width))
         if self.sink_name is not None:
             t[self.sink_name] = TensorSpec((self.H,), "vector")
+        if self.bias_name is not None:
+            t[self.bias_name] = TensorSpec((32, self.H), "vector", any_rows=True)
+        if self.value_share is not None:
+            # (the layer that leaves its values has no use for the number; a checkpoint may carry one)
+            t[self.v_mix_name] = TensorSpec((), "vector", optional=self.value_share == "first")
         return t
 
     def bind(self, tensors, rt):
@@ -150,6 +176,13 @@ class GQAAttention(Mixer):
             self.sink = tensors[self.sink_name].to(torch.float32).contiguous()
         elif self.sink_value is not None:
             self.sink = torch.full((self.H,), self.sink_value, dtype=torch.float32, device=rt.device)
+        if self.bias_name is not None:
+            rel = tensors[self.bias_name].to(torch.float32)                                   # [rows, H]
+            rows = torch.from_numpy(DistanceBuckets(rel.shape[0], self.bias_far).table()).to(rel.device)
+            # a row per head over distances, in units of the unscaled score, as the attention kernels take it
+            self.dist_bias = (rel[rows].t() / self.scale).contiguous()
+        if self.value_share == "mix":
+            self.v_lambda = float(tensors[self.v_mix_name].to(torch.float32).reshape(()).item())
         if self.value_rotation is not None:
             vf = np.power(float(self.value_rotation[0]), -2.0 * np.arange(self.Vd // 2, dtype=np.float64) / float(self.Vd))
             self.vfreq64 = torch.from_numpy(vf).to(rt.device)
@@ -212,12 +245,14 @@ class GQAAttention(Mixer):
             if self.value_rotation is not None:
                 kernels.rotate_heads(proj, (self.H + self.K) * self.D, self.K, self.Vd, self.Vd, self.Vd, self.value_rotation[1] == "adjacent",
                                      self.vfreq64, ctx.positions)
+            v_first = ctx.buf("shared_values", (n, self.K * self.Vd), ctx.act_dtype) if self.value_share is not None else None
             coef, every = self.q_temp if self.q_temp is not None else (0.0, 0)
             kernels.qk_norm_rope_store(proj, qkv, ctx.positions, ctx.tok_seg, bt, self.freq64, self.q_norm_w, self.k_norm_w, store_ptr,
                                        page_stride, v_offset, self.H, self.K, self.D, self.Vd, self.hd, rot_dim, ctx.max_pages,
                                        ctx.page_size, adjacent, self.norm_eps, self.unit_norm, coef, every,
                                        partial=None if pend is None else pend.partial, splits=0 if pend is None else pend.splits,
-                                       bias=None if pend is None else pend.bias, mscale=mscale, norm_after=self.norm_after)
+                                       bias=None if pend is None else pend.bias, mscale=mscale, norm_after=self.norm_after,
+                                       v_first=v_first, v_lambda=self.v_lambda)
             if pend is not None:
                 pend.release()
         else:
@@ -249,7 +284,8 @@ class GQAAttention(Mixer):
                 # prompt portions: S = Q K^T and O += P V on tcgen05
                 kernels.attention_tc(qkv, o, ctx.seg_start, ctx.seg_len, ctx.seg_pos0, bt, ctx.cache_group(lay), self.H,
                                      self.K, self.hd, ctx.max_pages, ctx.page_size, self.window or 0, self.scale, ctx.n_seg,
-                                     longest, row_tiles=tiles_tc, sink=self.sink, softcap=self.softcap)
+                                     longest, row_tiles=tiles_tc, sink=self.sink, softcap=self.softcap, keep_first=self.keep_first,
+                                     bias=self.dist_bias)
                 counters["tcgen05"] += 1
                 any_long = False
             if any_short or any_long:
@@ -257,11 +293,13 @@ class GQAAttention(Mixer):
                                       page_stride, v_offset, self.H, self.K, self.hd, ctx.max_pages, ctx.page_size,
                                       self.window or 0, self.scale, ctx.n_seg, longest, ctx.max_kv_len, splits,
                                       any_short, any_long, group=ctx.cache_group(lay) if USE_TMA else None, uneven=ctx.uneven,
-                                      row_tiles=tiles_rows, sink=self.sink, softcap=self.softcap)
+                                      row_tiles=tiles_rows, sink=self.sink, softcap=self.softcap, keep_first=self.keep_first,
+                                      bias=self.dist_bias)
                 counters["mma"] += 1
         else:
             kernels.attention_simt(qkv, qkv_dim, o, k_ptr, ctx.positions, ctx.tok_seg, bt, page_stride, v_offset,
-                                   self.H, self.K, self.hd, ctx.max_pages, ctx.page_size, self.window or 0, self.scale, sink=self.sink, softcap=self.softcap)
+                                   self.H, self.K, self.hd, ctx.max_pages, ctx.page_size, self.window or 0, self.scale, sink=self.sink, softcap=self.softcap,
+                                   keep_first=self.keep_first, bias=self.dist_bias)
             counters["simt"] += 1
         if self.gate is not None:
             kernels.sigmoid_gate(o, proj[:, gate_at:gate_at + self.gate_cols], self.H, self.hd, self.Vd, self.gate == "each")

@@ -58,6 +58,7 @@ class KVNeed:
     head_dim: int
     window: Optional[int] = None    # None: all keys; w: the last w keys
     planes: int = 2                 # arrays per token: 2 (keys and values), 1 for a mixer that caches one row per token
+    keep_first: int = 0             # with a window: a request's first keys that stay visible behind it
 
 
 @dataclass(frozen=True)

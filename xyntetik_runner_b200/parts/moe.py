@@ -3,7 +3,11 @@
     z = W_router h (float32);  the `top` experts with the largest z;  weights = softmax over the chosen z alone
     out = sum_j weight_j * expert_{e_j}(h)  (+ shared(h))
     expert(h) = W_down gate_act(W_gate h, W_up h), no biases
-With ``scoring="sigmoid"`` the scores are s = sigmoid(z); the `top` largest s + correction are chosen (`correction`: a tensor of
+With ``scoring="softmax_all"`` the scores are s = softmax(z) over all outputs of the router, which may have `identity` outputs
+more than there are experts: these identity experts take part in the choice like the others, their output is h itself, and
+they have no tensors.  The choice goes by s + correction; `groups=(count, keep)` splits the outputs into `count` equal groups of
+neighbours of which only the `keep` with the largest s + correction can be chosen from; the weights are s * `scale`, not
+renormalised.  With ``scoring="sigmoid"`` the scores are s = sigmoid(z); the `top` largest s + correction are chosen (`correction`: a tensor of
 one number per expert, or None) and the weights are the chosen experts' s, not renormalised.
 The activation is one of ``kernels.ACTIVATIONS`` (with its `limit` where it has one).  Experts' matrices are kept as
 [experts, rows, columns] arrays; the (token, choice) pairs are put in the order of their experts on the device and every
@@ -29,25 +33,32 @@ class RoutedExperts(FeedForward):
     def __init__(self, width: int, experts: int, top: int, inner: int, prefix: str, activation: str = "silu",
                  limit: float = 0.0, shared: Optional[GatedFeedForward] = None, router: str = "router",
                  expert: str = "e{}.", gate: str = "gate", up: str = "up", down: str = "down", scoring: str = "softmax",
-                 correction: Optional[str] = None):
-        if scoring not in ("softmax", "sigmoid"):
-            raise ValueError(f"{prefix}: scoring is 'softmax' (over the chosen logits) or 'sigmoid'")
-        if correction is not None and scoring != "sigmoid":
-            raise ValueError(f"{prefix}: a correction of the choice goes with sigmoid scores")
-        if not (1 <= top <= experts):
-            raise ValueError(f"{prefix}: top {top} of {experts} experts")
+                 correction: Optional[str] = None, identity: int = 0, groups: tuple = (1, 1), scale: float = 1.0):
+        if scoring not in ("softmax", "softmax_all", "sigmoid"):
+            raise ValueError(f"{prefix}: scoring is 'softmax' (over the chosen logits), 'softmax_all' or 'sigmoid'")
+        if correction is not None and scoring == "softmax":
+            raise ValueError(f"{prefix}: a correction of the choice goes with sigmoid scores or those of a softmax over all outputs")
+        if scoring != "softmax_all" and (identity or tuple(groups) != (1, 1) or float(scale) != 1.0):
+            raise ValueError(f"{prefix}: identity experts, groups and a factor on the weights go with scoring='softmax_all'")
+        count, keep = (int(g) for g in groups)
+        outputs = experts + int(identity)
+        if count < 1 or outputs % count or not (1 <= keep <= count):
+            raise ValueError(f"{prefix}: {outputs} outputs of the router in {count} groups of which {keep} are kept")
+        if not (1 <= top <= keep * (outputs // count)):
+            raise ValueError(f"{prefix}: top {top} of {keep * (outputs // count)} experts that can be chosen")
         self.width, self.E, self.top, self.inner, self.prefix = width, experts, top, inner, prefix
         self.act, self.limit, self.shared = _act_id(activation), float(limit), shared
         self.router_name = prefix + router
+        self.outputs, self.groups, self.scale, self.softmax_all = outputs, (count, keep), float(scale), scoring == "softmax_all"
         self.sigmoid, self.correction_name, self.correction = scoring == "sigmoid", None if correction is None else prefix + correction, None
         self.expert_names = [tuple(prefix + expert.format(e) + s for s in (gate, up, down)) for e in range(experts)]
         self.router = self.w_gate_up = self.w_down = None
         self.tensor_cores, self._nbytes = False, 0
 
     def tensors(self):
-        t = {self.router_name: TensorSpec((self.E, self.width))}
+        t = {self.router_name: TensorSpec((self.outputs, self.width))}
         if self.correction_name is not None:
-            t[self.correction_name] = TensorSpec((self.E,), "vector", "zeros")
+            t[self.correction_name] = TensorSpec((self.outputs,), "vector", "zeros")
         for g, u, d in self.expert_names:
             t[g] = TensorSpec((self.inner, self.width))
             t[u] = TensorSpec((self.inner, self.width))
@@ -92,11 +103,13 @@ class RoutedExperts(FeedForward):
     def forward(self, ctx, h, x):
         n, top, E = h.shape[0], self.top, self.E
         pairs = n * top
-        z = ctx.buf("moe_logits", (n, E), torch.float32)
+        z = ctx.buf("moe_logits", (n, self.outputs), torch.float32)
         self.router.forward(h, z)
         ids = ctx.buf("moe_ids", (n, top), torch.int32)
         wts = ctx.buf("moe_weights", (n, top), torch.float32)
-        if self.sigmoid:
+        if self.softmax_all:
+            kernels.route_groups(z, ids, wts, top, self.correction, *self.groups, self.scale)
+        elif self.sigmoid:
             kernels.route_topk(z, ids, wts, top, sigmoid_scores=True, correction=self.correction)
         else:
             kernels.route_topk(z, ids, wts, top)
@@ -118,7 +131,7 @@ class RoutedExperts(FeedForward):
             kernels.moe_gemm(h, self.w_gate_up, y, row_src, tile_group, top, True, self.act, self.limit)
             kernels.moe_gemm(y, self.w_down, zz, row_src, tile_group, top, False)
         ctx.materialize(x)
-        kernels.moe_combine(x, zz, wts, pair_row, top)
+        kernels.moe_combine(x, zz, wts, pair_row, top, h if self.outputs > E else None)
         if self.shared is not None:
             self.shared.forward(ctx, h, x)
 

@@ -13,6 +13,7 @@ kernel that also stores K and V.
 from __future__ import annotations
 
 import math
+from fractions import Fraction
 from typing import Optional
 
 import numpy as np
@@ -34,6 +35,37 @@ def llama3_divisors(inv_freq: np.ndarray, factor: float, low: float, high: float
             d = f / ((1.0 - s) * f / factor + s * f)
         out[j] = np.float32(d)
     return out
+
+
+class DistanceBuckets:
+    """Which row of a bias table of `rows` rows a distance from query to key takes: the distance itself below h = rows // 2, then
+    steps that grow logarithmically up to the distance `far`, the last row from there on,
+        min(rows - 1, h + floor(ln(n / h) / ln(far / h) (rows - h)))       for n >= h.
+    ``table()`` lists the rows of the distances 0, 1, ... up to the first that takes the last row (which every larger one takes too)."""
+
+    def __init__(self, rows: int, far: float):
+        self.rows, self.far, self.half = int(rows), Fraction(far), int(rows) // 2
+        if self.half < 1 or self.far <= self.half:
+            raise ValueError(f"distance buckets: {rows} rows up to the distance {far}: at least two rows, and a distance above half of them")
+
+    def _start(self, k: int) -> int:
+        """The first distance of step k: the smallest n with (n / h)^steps >= (far / h)^k, compared in whole numbers, so that a
+        distance right on a step takes it."""
+        h, steps = self.half, self.rows - self.half
+        reached = lambda n: Fraction(n, h) ** steps >= (self.far / h) ** k
+        n = max(h, int(h * float(self.far / h) ** (k / steps)))
+        while not reached(n):
+            n += 1
+        while n > h and reached(n - 1):
+            n -= 1
+        return n
+
+    def table(self) -> np.ndarray:
+        h, steps = self.half, self.rows - self.half
+        starts = np.asarray([self._start(k) for k in range(1, steps)], dtype=np.int64)     # (the last row is rows - 1 = h + steps - 1)
+        last = int(starts[-1]) if len(starts) else h
+        n = np.arange(last + 1, dtype=np.int64)
+        return np.where(n < h, n, h + np.searchsorted(starts, n, side="right"))
 
 
 class Rope(PositionEncoding):

@@ -31,6 +31,7 @@ class TensorSpec:
     kind: str = "matrix"          # "matrix" | "vector" | "table" (integers)
     init: str = "normal"          # random mode: "normal" | "ones" | "ones_jitter" | "zeros" | "zeros_jitter"
     optional: bool = False        # a source may lack it (the model then never reads it); random sources leave it out
+    any_rows: bool = False        # the source says how many rows there are; shape[0] is what random sources make
 
 
 class WeightsError(ValueError):
@@ -163,7 +164,10 @@ def load_tensors(expected: Mapping[str, TensorSpec], source: TensorSource,
         if n not in have:
             continue
         dt, shape = have[n]
-        if tuple(shape) != tuple(spec.shape):
+        same = tuple(shape) == tuple(spec.shape)
+        if spec.any_rows:
+            same = len(shape) == len(spec.shape) and shape[0] >= 1 and tuple(shape[1:]) == tuple(spec.shape[1:])
+        if not same:
             wrong.append((n, tuple(shape), tuple(spec.shape)))
         if spec.kind == "table":
             if dt not in (torch.int32, torch.int64):
