@@ -73,6 +73,36 @@ def test_window_group_releases_pages_behind_the_window():
     m.audit()
 
 
+def test_kept_first_pages_stay_behind_the_window():
+    """Window 6, first 5 positions kept, pages of 4: pages 0 and 1 stay to the end, pages between them and the window go."""
+    m = CacheManager([GroupSpec("w", window=6, keep_first=5)], n_pages=6, page_size=4, max_requests=2, max_request_tokens=400)
+    m.open("a")
+    held = lambda: [i for i, p in enumerate(m.block_table(0, "a")) if p >= 0]
+    first = None
+    for n in range(100):
+        m.reserve("a", 1); m.commit("a")
+        m.audit()
+        lo = max(0, n - 6 + 1) // 4
+        assert held() == sorted({i for i in (0, 1) if i <= n // 4} | set(range(lo, n // 4 + 1))), n
+        first = first if first is not None else m.block_table(0, "a")[0]
+        assert m.block_table(0, "a")[0] == first                # the same page all along
+        # what a reservation would take and what is free agree with what it then takes
+        need, free = m.pages_needed("a", 3), m.free_pages()
+        m.reserve("a", 3); m.audit(); m.cancel("a"); m.audit()
+        assert need == [(n + 4 + 3) // 4 - (n + 4) // 4] and m.free_pages()[0] >= free[0]
+    m.open("b"); m.reserve("b", 3); m.commit("b")                # shorter than the kept positions
+    m.audit()
+    m.close("a"); m.close("b")
+    assert m.free_pages() == [6]
+    m.audit()
+    # kept positions that fill the pool leave no room behind them
+    m.open("c"); m.reserve("c", 24); m.commit("c")
+    with pytest.raises(OutOfPages):
+        m.reserve("c", 12)
+    m.reserve("c", 8)                                            # pages 2 and 3 lie behind the window of position 24
+    m.audit()
+
+
 def test_window_lets_a_long_request_live_in_a_small_pool():
     m = CacheManager([GroupSpec("w", window=5)], n_pages=4, page_size=4, max_requests=1, max_request_tokens=400)
     m.open("a")
@@ -164,14 +194,16 @@ def test_describe_step_flattens_a_batch():
         m.describe_step(slots, counts, tokens, want_counts, wants, 0, 16, [a.ctypes.data for a in arrs], [b.ctypes.data for b in bts])
 
 
-@pytest.mark.parametrize("seed", range(4))
+@pytest.mark.parametrize("seed", range(8))
 def test_pages_held_follow_the_formula(seed):
     """After every commit a request holds, in a group that keeps all keys, ceil(length / page) pages, and in a window
-    group the pages from the one that holds the first key its next query can still read up to the last: counted here
-    from lengths alone and compared with the pools."""
+    group the pages from the one that holds the first key its next query can still read up to the last, and those of the kept
+    first positions: counted here from lengths alone and compared with the pools."""
     rng = np.random.RandomState(50 + seed)
     ps, window, n_pages = int(rng.choice([2, 4, 8])), int(rng.randint(2, 30)), 200
-    m = CacheManager([GroupSpec("full"), GroupSpec("w", window=window)], n_pages, ps, 5, ps * 30)
+    keep = int(rng.randint(1, 20)) if seed >= 4 else 0
+    m = CacheManager([GroupSpec("full"), GroupSpec("w", window=window, keep_first=keep)], n_pages, ps, 5, ps * 30)
+    kept = -(-keep // ps)
     lengths = {}
 
     released = {}                                   # request -> first page index still held in the window group
@@ -193,9 +225,10 @@ def test_pages_held_follow_the_formula(seed):
             rid = list(lengths)[rng.randint(len(lengths))]
             m.close(rid); del lengths[rid]; del released[rid]
         full = sum(-(-n // ps) for n in lengths.values())
-        win = sum(-(-n // ps) - released[rid] for rid, n in lengths.items())
+        win = sum(-(-n // ps) - max(0, released[rid] - kept) for rid, n in lengths.items())
         assert m.free_pages() == [n_pages - full, n_pages - win], (it, lengths, released)
         for rid, n in lengths.items():
             tab = m.block_table(1, rid)
-            assert (tab[:released[rid]] == -1).all() and (tab[released[rid]:-(-n // ps)] >= 0).all()
+            assert (tab[kept:max(kept, released[rid])] == -1).all() and (tab[max(kept, released[rid]):-(-n // ps)] >= 0).all()
+            assert (tab[:min(kept, -(-n // ps))] >= 0).all() and (tab[-(-n // ps):] == -1).all()
     m.audit()
