@@ -1,5 +1,6 @@
-"""Prefill and decode throughput of a Turudra, a Besolix, a Pitolix or a Buzarax model beside a dense Llama of equal size, with the time of
-every kernel family inside the steps (``bench.py --designs``).
+"""Prefill and decode throughput of a Turudra, a Besolix, a Pitolix, a Buzarax or a Semesun model beside a dense Llama of equal size (Semesun:
+also beside a Buzarax model, whose recurrences and experts are the nearest to its own), with the time of every kernel family inside the
+steps (``bench.py --designs``).
 
 Sizes resemble real layers; weights are random.  Both models run through the same engine: one prompt of `tokens` tokens
 in one step (prefill), and decode steps of `batch` requests that hold `context` tokens each (``Engine.adopt``: the cache
@@ -23,6 +24,7 @@ from .config.besolix import BesolixConfig
 from .config.buzarax import BuzaraxConfig
 from .config.llama import LlamaConfig
 from .config.pitolix import PitolixConfig
+from .config.semesun import SemesunConfig
 from .config.turudra import TurudraConfig
 from .engine.engine import EngineParams, StepEntry, random_engine
 
@@ -149,6 +151,36 @@ def llama_like_buzarax(size: str, positions: int) -> LlamaConfig:
                                   "max_position_embeddings": positions, "torch_dtype": "bfloat16"})
 
 
+SEMESUN_SIZES = {
+    # name: (width, attention (heads, kv heads, head size, window, kept tokens, reach of the bias), recurrence (heads, value size, state,
+    # groups, taps), dense feed-forward, experts, identity experts, chosen, groups, groups kept, expert feed-forward, vocab); six layers:
+    # attention and the recurrence in turn, dense and routed feed-forwards in turn
+    "semesun-w1024": (1024, (8, 2, 128, 1024, 4, 512), (32, 64, 128, 1, 4), 4096, 12, 4, 2, 4, 2, 1408, 32000),
+    "semesun-w2048": (2048, (16, 4, 128, 1024, 4, 512), (64, 64, 128, 1, 4), 8192, 12, 4, 2, 4, 2, 2816, 32000),
+}
+
+
+def semesun_config(size: str) -> SemesunConfig:
+    W, (H, K, D, window, keep, far), (mh, mv, mn, mg, taps), ff, E, identity, top, groups, kept, eff, vocab = SEMESUN_SIZES[size]
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "router": {"experts": E, "identity": identity, "top": top, "groups": {"count": groups, "keep": kept}, "scale": 2.0},
+           "expert": {"ff": eff, "limit": 7.0}}
+    att = {"type": "attention", "mixer": {"heads": H, "kv_heads": K, "dim": D, "vdim": D, "scale": D ** -0.5, "bias_max": far, "v_mix": True,
+                                          "mask": {"size": window, "keep_first": keep}}}
+    rec = {"type": "mamba2", "mixer": {"heads": mh, "vdim": mv, "state": mn, "groups": mg, "conv": taps, "norm_groups": 1}}
+    layers = [dict(att, mlp=dense), dict(rec, mlp=moe), dict(att, mlp=moe), dict(rec, mlp=dense), dict(att, mlp=dense), dict(rec, mlp=moe)]
+    return SemesunConfig.from_dict({"architecture": "Semesun", "vocab": vocab, "width": W, "norm": {"eps": 1e-5}, "layers": layers})
+
+
+def llama_like_semesun(size: str, positions: int) -> LlamaConfig:
+    """A dense decoder of the same width, number of layers, attention heads and window, its feed-forward about as wide as what a token uses."""
+    W, (H, K, D, window, keep, far), _, ff, E, identity, top, groups, kept, eff, vocab = SEMESUN_SIZES[size]
+    return LlamaConfig.from_dict({"architectures": ["LlamaForCausalLM"], "hidden_size": W, "num_hidden_layers": 6,
+                                  "num_attention_heads": H, "num_key_value_heads": K, "head_dim": D, "intermediate_size": top * eff,
+                                  "vocab_size": vocab, "rms_norm_eps": 1e-5, "rope_theta": 10000.0, "sliding_window": window,
+                                  "max_position_embeddings": positions, "torch_dtype": "bfloat16"})
+
+
 FAMILIES = {
     "gemm_tc": "products (tcgen05)", "gemm_tc_deferred": "products (tcgen05)", "gemm_simt": "products (FMA)",
     "finish_plain": "products (tcgen05)", "finish_add_rmsnorm": "norms", "rmsnorm": "norms", "finish_rope_store": "rotation + cache store",
@@ -159,7 +191,7 @@ FAMILIES = {
     "heads_scatter_gate": "grouped products (experts, per-head)",
     "mlstm": "mlstm recurrence", "route_topk": "routing", "moe_plan": "routing", "moe_gemm": "experts' products", "moe_combine": "experts' sum",
     "delta": "delta recurrence", "head_norm_gate": "delta recurrence", "qk_norm_rope_store": "rotation + cache store",
-    "rmsnorm_act": "norms",
+    "rmsnorm_act": "norms", "ssd": "state-space recurrence", "silu_gate_norm": "gated norm of the recurrence", "route_groups": "routing",
     "sigmoid_gate": "output gates", "stream_step": "stream kernels",
     "rglru": "gated linear recurrence", "decay_attention": "decay attention recurrence", "norm_add": "norms", "depth_average": "stream kernels",
     "cast_rows": "stream kernels", "row_norm_gate": "decay attention recurrence", "embed_pair": "stream kernels", "last_token": "stream kernels", "rotate_heads": "rotation + cache store",
@@ -341,6 +373,72 @@ def _buzarax_work(cfg, tokens, keys_per_token, decode):
             "stream kernels": (0.0, by_s)}
 
 
+def _window_keys(tokens: int, keys_per_token: float, window, keep: int, decode: bool) -> float:
+    """Keys that a token of the step sees on average: in a prompt from its first token on, the token at position i min(i + 1, window)."""
+    if not window:
+        return keys_per_token
+    if decode:
+        return min(keys_per_token, window + keep)
+    full = min(tokens, window)
+    return (full * (full + 1) / 2.0 + (tokens - full) * window + keep * max(0, tokens - window - keep)) / tokens
+
+
+def _llama_window_work(cfg, tokens, keys_per_token, decode):
+    """``_llama_work`` with the window's keys counted exactly."""
+    work = _llama_work(cfg, tokens, keys_per_token, decode)
+    keys = _window_keys(tokens, keys_per_token, cfg.sliding_window, 0, decode)
+    L, once = cfg.num_hidden_layers, tokens if decode else 1
+    work["attention"] = (4.0 * tokens * cfg.num_attention_heads * keys * cfg.head_dim * L,
+                         once * (keys if decode else tokens) * 2 * cfg.num_key_value_heads * cfg.head_dim * 2 * L)
+    return work
+
+
+def _semesun_work(cfg, tokens, keys_per_token, decode):
+    """(FLOPs, bytes) per kernel family in one step of `tokens` tokens, counted like ``_llama_work``."""
+    W = cfg.width
+    fl_a = by_a = fl_p = by_p = by_n = by_r = fl_s = by_s = by_g = fl_e = by_e = by_c = 0.0
+    once = tokens if decode else 1
+    for lay in cfg.layers:
+        m = lay.mixer
+        if m.kind == "attention":
+            hd = max(m.dim, m.vdim)
+            keys = _window_keys(tokens, keys_per_token, m.window, m.keep_first, decode)
+            cols = (m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim
+            per = W * cols + m.heads * m.vdim * W
+            fl_a += 2.0 * tokens * m.heads * keys * (m.dim + m.vdim)
+            by_a += once * (keys if decode else tokens) * 2 * m.kv_heads * hd * 2
+            # the norm/store kernel; the shared values are written or read with it
+            by_r += tokens * 2.0 * (cols + (m.heads + 2 * m.kv_heads) * hd + (m.kv_heads * m.vdim if m.v_mix else 0))
+        else:
+            inner = m.heads * m.vdim
+            ch = inner + 2 * m.groups * m.state
+            per = W * (inner + ch + m.heads) + inner * W
+            # per token and state element: decay and update, read-out; the state once per request and step; the convolution reads and
+            # writes its channels, the walk reads them and writes its read-outs, in float32
+            fl_s += 4.0 * tokens * inner * m.state
+            by_s += once * 2 * inner * m.state * 4 + tokens * 4.0 * (3 * ch + inner + 3 * m.heads)
+            by_g += tokens * inner * (4 + 4 + 2.0)
+        f = lay.mlp
+        if f is not None and f.kind == "dense":
+            per += 2 * W * f.ff
+        elif f is not None:
+            # of the chosen outputs a share are identity experts, which multiply nothing; a third pass adds the pairs' rows
+            real = f.top * f.experts / (f.experts + f.identity)
+            fl_e += 2.0 * tokens * real * 3 * f.ff * W
+            by_e += min(f.experts, tokens * real) * 3 * f.ff * W * 2
+            by_c += tokens * W * 4.0 * (real + 2) + tokens * W * 2.0
+            per += (f.experts + f.identity) * W
+        fl_p += 2.0 * tokens * per
+        by_p += 2.0 * per
+        by_n += tokens * W * (4 + 2) * (2 if f is not None else 1)
+    fl_p += 2.0 * cfg.vocab * W * (tokens if decode else 1)
+    by_p += 2.0 * cfg.vocab * W
+    by_n += tokens * W * (4 + 2)
+    return {"attention": (fl_a, by_a), "products (tcgen05)": (fl_p, by_p), "norms": (0.0, by_n), "rotation + cache store": (0.0, by_r),
+            "state-space recurrence": (fl_s, by_s), "gated norm of the recurrence": (0.0, by_g), "grouped products (experts, per-head)": (fl_e, by_e),
+            "experts' sum": (0.0, by_c)}
+
+
 def _measure(eng, cfg, work_fn, tokens: int, batch: int, context: int, steps: int, warmup: int, pk, phase: str = "both") -> dict:
     vocab = eng.plan.vocab_size
     gen = torch.Generator().manual_seed(0)
@@ -427,7 +525,11 @@ def compare(size: str, tokens: int = 2048, batch: int = 8, context: int = 2048, 
     pool = batch * (context + 64 * (2 + (steps + warmup + 8) // 64)) + tokens + 64
     ep = lambda: EngineParams(dtype="bfloat16", max_tokens=pool, page_size=64, max_requests=batch + 1,
                               max_request_tokens=max(tokens, context + steps + warmup + 72), max_step_tokens=tokens)
-    if size in BUZARAX_SIZES:
+    if size in SEMESUN_SIZES:
+        near = size.replace("semesun", "buzarax")
+        arms = (("semesun", semesun_config(size), _semesun_work), ("buzarax", buzarax_config(near), _buzarax_work),
+                ("llama", llama_like_semesun(size, context + tokens), _llama_window_work))
+    elif size in BUZARAX_SIZES:
         arms = (("buzarax", buzarax_config(size), _buzarax_work), ("llama", llama_like_buzarax(size, context + tokens), _llama_work))
     elif size in PITOLIX_SIZES:
         arms = (("pitolix", pitolix_config(size), _pitolix_work), ("llama", llama_like_pitolix(size, context + tokens), _llama_work))
@@ -438,7 +540,7 @@ def compare(size: str, tokens: int = 2048, batch: int = 8, context: int = 2048, 
         arms = (("turudra", tcfg, _work), ("llama", llama_config(size, len(tcfg.layer_runs()), context + tokens), _llama_work))
     for name, cfg, work in arms:
         # (`models` names arms to run; "turudra" also stands for the new design's arm of a Besolix size: the default runs both arms)
-        if name not in models and not (name in ("besolix", "pitolix", "buzarax") and "turudra" in models):
+        if name not in models and not (name in ("besolix", "pitolix", "buzarax", "semesun") and "turudra" in models):
             continue
         t0 = time.perf_counter()
         eng = random_engine(cfg, 5, ep())
