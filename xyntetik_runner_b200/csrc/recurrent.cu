@@ -453,54 +453,60 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
         for (int t0 = 0; t0 < here; t0 += TB) {
             float acc[TB * VC];
 #pragma unroll
-            for (int tb = 0; tb < TB; tb++) {
+            for (int k = 0; k < TB * VC; k++) acc[k] = 0.f;
+            auto token = [&](int tb) {
+                const float* row = base + (t0 + tb) * RW;
+                float q[JD], k[JD], v[VC];
+                float a = dec;
+                if constexpr (JD % 4 == 0) {
 #pragma unroll
-                for (int c = 0; c < VC; c++) acc[tb * VC + c] = 0.f;
-                if (t0 + tb < here) {
-                    const float* row = base + (t0 + tb) * RW;
-                    float q[JD], k[JD], v[VC];
-                    float a = dec;
-                    if constexpr (JD % 4 == 0) {
-#pragma unroll
-                        for (int j = 0; j < JD; j += 4) {
-                            const float4 a = *reinterpret_cast<const float4*>(row + lane * JD + j);
-                            const float4 b = *reinterpret_cast<const float4*>(row + DP + lane * JD + j);
-                            q[j] = a.x; q[j + 1] = a.y; q[j + 2] = a.z; q[j + 3] = a.w;
-                            k[j] = b.x; k[j + 1] = b.y; k[j + 2] = b.z; k[j + 3] = b.w;
-                        }
-                    } else if constexpr (JD == 2) {
-                        const float2 a = *reinterpret_cast<const float2*>(row + lane * 2);
-                        const float2 b = *reinterpret_cast<const float2*>(row + DP + lane * 2);
-                        q[0] = a.x; q[1] = a.y; k[0] = b.x; k[1] = b.y;
-                    } else {
-#pragma unroll
-                        for (int j = 0; j < JD; j++) { q[j] = row[lane * JD + j]; k[j] = row[DP + lane * JD + j]; }
+                    for (int j = 0; j < JD; j += 4) {
+                        const float4 a = *reinterpret_cast<const float4*>(row + lane * JD + j);
+                        const float4 b = *reinterpret_cast<const float4*>(row + DP + lane * JD + j);
+                        q[j] = a.x; q[j + 1] = a.y; q[j + 2] = a.z; q[j + 3] = a.w;
+                        k[j] = b.x; k[j + 1] = b.y; k[j + 2] = b.z; k[j + 3] = b.w;
                     }
-                    if constexpr (VC % 4 == 0) {
+                } else if constexpr (JD == 2) {
+                    const float2 a = *reinterpret_cast<const float2*>(row + lane * 2);
+                    const float2 b = *reinterpret_cast<const float2*>(row + DP + lane * 2);
+                    q[0] = a.x; q[1] = a.y; k[0] = b.x; k[1] = b.y;
+                } else {
 #pragma unroll
-                        for (int c = 0; c < VC; c += 4) {
-                            const float4 a = *reinterpret_cast<const float4*>(row + 2 * DP + warp * VC + c);
-                            v[c] = a.x; v[c + 1] = a.y; v[c + 2] = a.z; v[c + 3] = a.w;
-                        }
-                    } else {
+                    for (int j = 0; j < JD; j++) { q[j] = row[lane * JD + j]; k[j] = row[DP + lane * JD + j]; }
+                }
+                if constexpr (VC % 4 == 0) {
 #pragma unroll
-                        for (int c = 0; c < VC; c++) v[c] = row[2 * DP + warp * VC + c];
+                    for (int c = 0; c < VC; c += 4) {
+                        const float4 a = *reinterpret_cast<const float4*>(row + 2 * DP + warp * VC + c);
+                        v[c] = a.x; v[c + 1] = a.y; v[c + 2] = a.z; v[c + 3] = a.w;
                     }
-                    if constexpr (SSD) {
-                        const float2 ad = *reinterpret_cast<const float2*>(da_coef + ((ch & 1) * CH + t0 + tb) * 2);
-                        a = ad.x;
+                } else {
 #pragma unroll
-                        for (int c = 0; c < VC; c++) v[c] *= ad.y;
-                    }
+                    for (int c = 0; c < VC; c++) v[c] = row[2 * DP + warp * VC + c];
+                }
+                if constexpr (SSD) {
+                    const float2 ad = *reinterpret_cast<const float2*>(da_coef + ((ch & 1) * CH + t0 + tb) * 2);
+                    a = ad.x;
 #pragma unroll
-                    for (int j = 0; j < JD; j++) {
+                    for (int c = 0; c < VC; c++) v[c] *= ad.y;
+                }
 #pragma unroll
-                        for (int c = 0; c < VC; c++) {
-                            s[c][j] = fmaf(a, s[c][j], k[j] * v[c]);
-                            acc[tb * VC + c] = fmaf(s[c][j], q[j], acc[tb * VC + c]);
-                        }
+                for (int j = 0; j < JD; j++) {
+#pragma unroll
+                    for (int c = 0; c < VC; c++) {
+                        s[c][j] = fmaf(a, s[c][j], k[j] * v[c]);
+                        acc[tb * VC + c] = fmaf(s[c][j], q[j], acc[tb * VC + c]);
                     }
                 }
+            };
+            // (a whole batch of tokens without a branch between them: their reads of shared memory are then in flight together)
+            if (t0 + TB <= here) {
+#pragma unroll
+                for (int tb = 0; tb < TB; tb++) token(tb);
+            } else {
+#pragma unroll
+                for (int tb = 0; tb < TB; tb++)
+                    if (t0 + tb < here) token(tb);
             }
             // 32 sums a lane -> one: a lane whose bit is set keeps the upper half of what it carries and hands over the lower one
 #pragma unroll

@@ -211,7 +211,7 @@ XR_EXPORT int xr_row_norm_gate(const float* o, const float* g, long long ld_g, c
 __device__ __forceinline__ float st_silu_gated(float o, float g) { return o * (g < -80.0f ? 0.0f : g / (1.0f + expf(-g))); }
 
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(1024)
 k_silu_gate_norm(const float* __restrict__ o, const float* __restrict__ g, long long ld_g, const float* __restrict__ w, T* __restrict__ y,
                  int width, int per, float eps) {
     xr_pdl_launch();
@@ -243,7 +243,9 @@ k_silu_gate_norm(const float* __restrict__ o, const float* __restrict__ g, long 
 XR_EXPORT int xr_silu_gate_norm(const float* o, const float* g, long long ld_g, const float* w, void* y, int dtype, int n, int width, int groups,
                                 float eps, cudaStream_t stream) {
     if (n < 1 || width < 1 || groups < 1 || width % groups || groups > 65535) return XR_ERR_ARG;
-    const int per = width / groups, threads = per >= 256 ? 256 : (per + 31) / 32 * 32;
+    const int per = width / groups;
+    // (few rows: nothing but a row's own threads hides its loads' latency)
+    const int most = (long long)n * groups <= xr_sm_count() ? 1024 : 256, threads = per >= most ? most : (per + 31) / 32 * 32;
     const dim3 grid(n, groups);
     if (dtype == XR_F32) xr_launch((k_silu_gate_norm<float>), grid, dim3(threads), 0, stream, o, g, ld_g, w, (float*)y, width, per, eps);
     else if (dtype == XR_BF16) xr_launch((k_silu_gate_norm<__nv_bfloat16>), grid, dim3(threads), 0, stream, o, g, ld_g, w, (__nv_bfloat16*)y, width, per, eps);
