@@ -13,24 +13,9 @@ from ..config.registry import register_architecture
 from ..config.semesun import NAME, AttentionConfig, DenseConfig, ExpertsConfig, MambaConfig, SemesunConfig
 from ..engine.model import ModelPlan, ScheduleEntry
 from ..parts import MLP, Embedding, GQAAttention, Head, Mamba2, NoPosition, PreNormBlock, RMSNorm, RoutedExperts
-from ..weights.loader import TensorSpec
 
 # no position table limits a request's length: positions enter as distances only, and the recurrence has none
 MAX_POSITIONS = 1 << 30
-
-
-class _Block(PreNormBlock):
-    """A pre-norm layer; one without a feed-forward lets a checkpoint carry a second norm weight that nothing reads."""
-
-    def __init__(self, *parts, spare: str = None):
-        super().__init__(*parts)
-        self.spare = spare
-
-    def tensors(self):
-        out = super().tensors()
-        if self.spare is not None:
-            out[self.spare] = TensorSpec((self.mixer_norm.width,), kind="vector", init="ones", optional=True)
-        return out
 
 
 def build_semesun(cfg: SemesunConfig) -> ModelPlan:
@@ -52,7 +37,7 @@ def build_semesun(cfg: SemesunConfig) -> ModelPlan:
             raise ValueError(f"layer {i}: unknown mixer configuration {type(m).__name__}")
         norm1 = RMSNorm(W, eps, p + "norm1")
         if lay.mlp is None:
-            blocks.append(_Block(norm1, mixer, spare=p + "norm2"))
+            blocks.append(PreNormBlock(norm1, mixer, spare_norm=p + "norm2"))
         else:
             if isinstance(lay.mlp, DenseConfig):
                 ff = MLP(W, lay.mlp.ff, p + "mlp.", "relu2", up="up", down="down")
@@ -62,7 +47,7 @@ def build_semesun(cfg: SemesunConfig) -> ModelPlan:
                                    correction="correction", identity=f.identity, groups=(f.group_count, f.group_keep), scale=f.scale)
             else:
                 raise ValueError(f"layer {i}: unknown feed-forward configuration {type(lay.mlp).__name__}")
-            blocks.append(_Block(norm1, mixer, RMSNorm(W, eps, p + "norm2"), ff))
+            blocks.append(PreNormBlock(norm1, mixer, RMSNorm(W, eps, p + "norm2"), ff))
         schedule.append(ScheduleEntry(layer=i))
     return ModelPlan(embedding=Embedding(cfg.vocab, W, "embed"), blocks=blocks, schedule=schedule, final_norm=RMSNorm(W, eps, "final.norm"),
                      head=Head(cfg.vocab, W, name="head"), width=W, vocab_size=cfg.vocab, max_positions=MAX_POSITIONS)

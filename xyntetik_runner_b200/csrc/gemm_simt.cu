@@ -16,7 +16,7 @@
 template <typename TX, typename TW, typename TO, bool ACCUM>
 __global__ void __launch_bounds__(256)
 k_gemm_simt(const TX* __restrict__ X, const TW* __restrict__ W, const float* __restrict__ bias,
-            TO* __restrict__ out, int n, int n_out, int K, long long ldx, long long ldo) {
+            TO* __restrict__ out, int n, int n_out, int K, long long ldx, long long ldo, float alpha) {
     __shared__ float Xs[GS_BK][GS_BM + 4];
     __shared__ float Ws[GS_BK][GS_BN + 4];
     int tid = threadIdx.x;
@@ -60,7 +60,7 @@ k_gemm_simt(const TX* __restrict__ X, const TW* __restrict__ W, const float* __r
         for (int j = 0; j < 4; j++) {
             int r = r0 + tx * 4 + j;
             if (r >= n_out) continue;
-            float v = acc[i][j];
+            float v = alpha * acc[i][j];
             if (bias) v += bias[r];
             size_t o = (size_t)t * ldo + r;
             if (ACCUM) out[o] = xr_from_f32<TO>(xr_to_f32<TO>(out[o]) + v);
@@ -71,16 +71,16 @@ k_gemm_simt(const TX* __restrict__ X, const TW* __restrict__ W, const float* __r
 
 template <typename TX, typename TW>
 static int launch_simt(const void* X, const void* W, const float* bias, void* out, int out_dtype, int accumulate,
-                       int n, int n_out, int K, long long ldx, long long ldo, cudaStream_t stream) {
+                       int n, int n_out, int K, long long ldx, long long ldo, float alpha, cudaStream_t stream) {
     dim3 grid((n_out + GS_BN - 1) / GS_BN, (n + GS_BM - 1) / GS_BM);
     if (grid.y > 65535) return XR_ERR_ARG;
     if (accumulate) {
         if (out_dtype != XR_F32) return XR_ERR_ARG;
-        k_gemm_simt<TX, TW, float, true><<<grid, 256, 0, stream>>>((const TX*)X, (const TW*)W, bias, (float*)out, n, n_out, K, ldx, ldo);
+        k_gemm_simt<TX, TW, float, true><<<grid, 256, 0, stream>>>((const TX*)X, (const TW*)W, bias, (float*)out, n, n_out, K, ldx, ldo, alpha);
     } else if (out_dtype == XR_F32) {
-        k_gemm_simt<TX, TW, float, false><<<grid, 256, 0, stream>>>((const TX*)X, (const TW*)W, bias, (float*)out, n, n_out, K, ldx, ldo);
+        k_gemm_simt<TX, TW, float, false><<<grid, 256, 0, stream>>>((const TX*)X, (const TW*)W, bias, (float*)out, n, n_out, K, ldx, ldo, alpha);
     } else if (out_dtype == XR_BF16) {
-        k_gemm_simt<TX, TW, __nv_bfloat16, false><<<grid, 256, 0, stream>>>((const TX*)X, (const TW*)W, bias, (__nv_bfloat16*)out, n, n_out, K, ldx, ldo);
+        k_gemm_simt<TX, TW, __nv_bfloat16, false><<<grid, 256, 0, stream>>>((const TX*)X, (const TW*)W, bias, (__nv_bfloat16*)out, n, n_out, K, ldx, ldo, alpha);
     } else {
         return XR_ERR_ARG;
     }
@@ -88,14 +88,14 @@ static int launch_simt(const void* X, const void* W, const float* bias, void* ou
 }
 
 // X: [n, K] with row stride ldx; W: [n_out, K] dense; out: [n, n_out] with row stride ldo.
-// accumulate != 0 adds into a float32 `out` (the residual stream).
+// accumulate != 0 adds into a float32 `out` (the residual stream).  alpha multiplies every sum, ahead of the bias.
 XR_EXPORT int xr_gemm_simt(const void* X, int x_dtype, const void* W, int w_dtype, const float* bias, void* out,
                            int out_dtype, int accumulate, int n, int n_out, int K, long long ldx, long long ldo,
-                           cudaStream_t stream) {
+                           float alpha, cudaStream_t stream) {
     if (n < 1 || n_out < 1 || K < 1 || ldx < K || ldo < n_out) return XR_ERR_ARG;
-    if (x_dtype == XR_F32 && w_dtype == XR_F32) return launch_simt<float, float>(X, W, bias, out, out_dtype, accumulate, n, n_out, K, ldx, ldo, stream);
-    if (x_dtype == XR_F32 && w_dtype == XR_BF16) return launch_simt<float, __nv_bfloat16>(X, W, bias, out, out_dtype, accumulate, n, n_out, K, ldx, ldo, stream);
-    if (x_dtype == XR_BF16 && w_dtype == XR_F32) return launch_simt<__nv_bfloat16, float>(X, W, bias, out, out_dtype, accumulate, n, n_out, K, ldx, ldo, stream);
-    if (x_dtype == XR_BF16 && w_dtype == XR_BF16) return launch_simt<__nv_bfloat16, __nv_bfloat16>(X, W, bias, out, out_dtype, accumulate, n, n_out, K, ldx, ldo, stream);
+    if (x_dtype == XR_F32 && w_dtype == XR_F32) return launch_simt<float, float>(X, W, bias, out, out_dtype, accumulate, n, n_out, K, ldx, ldo, alpha, stream);
+    if (x_dtype == XR_F32 && w_dtype == XR_BF16) return launch_simt<float, __nv_bfloat16>(X, W, bias, out, out_dtype, accumulate, n, n_out, K, ldx, ldo, alpha, stream);
+    if (x_dtype == XR_BF16 && w_dtype == XR_F32) return launch_simt<__nv_bfloat16, float>(X, W, bias, out, out_dtype, accumulate, n, n_out, K, ldx, ldo, alpha, stream);
+    if (x_dtype == XR_BF16 && w_dtype == XR_BF16) return launch_simt<__nv_bfloat16, __nv_bfloat16>(X, W, bias, out, out_dtype, accumulate, n, n_out, K, ldx, ldo, alpha, stream);
     return XR_ERR_ARG;
 }

@@ -173,6 +173,7 @@ struct TcParams {
     // multiplies by matrix tile_group[t] (below zero: the tile holds no rows and its CTAs leave at once)
     const int* tile_group;
     int group_row_tiles;        // row tiles of one matrix in the packed array
+    float alpha = 1.f;          // factor on the accumulator, ahead of bias and activation (not for gated products)
 };
 
 // ---------------------------------------------------------------------------------------------
@@ -234,7 +235,7 @@ __device__ __forceinline__ void tc_epilogue(const TcParams& p, uint32_t tmem_bas
             for (int c = 0; c < 16; c++) xr_ld_fence(old[c]);
 #pragma unroll
             for (int c = 0; c < 16; c++)
-                if (tok0 + c0 + c < p.n) dst[(size_t)c * p.ldo] = old[c] + (g[c] + b);
+                if (tok0 + c0 + c < p.n) dst[(size_t)c * p.ldo] = old[c] + fmaf(p.alpha, g[c], b);
             continue;
         }
         // a chunk that runs past the last token stores only what exists
@@ -244,12 +245,12 @@ __device__ __forceinline__ void tc_epilogue(const TcParams& p, uint32_t tmem_bas
             float* dst = p.partial + ((size_t)split * p.n + tok0 + c0) * width + r;
 #pragma unroll
             for (int c = 0; c < 16; c++)
-                if (c < live) dst[(size_t)c * width] = g[c];
+                if (c < live) dst[(size_t)c * width] = p.alpha * g[c];
             continue;
         }
         float v[16];
 #pragma unroll
-        for (int c = 0; c < 16; c++) v[c] = tc_act(p.act, g[c] + b);
+        for (int c = 0; c < 16; c++) v[c] = tc_act(p.act, fmaf(p.alpha, g[c], b));
         if (p.out_dtype == XR_BF16) {
             __nv_bfloat16* dst = (__nv_bfloat16*)p.out + (size_t)(tok0 + c0) * p.ldo + r;
 #pragma unroll
@@ -806,7 +807,8 @@ XR_EXPORT long long xr_gemm_tc_scratch_floats(int n, int n_out, int gated) {
 // in each quarter sixteen gate rows, then their sixteen up rows); n_out counts features and out is [n, n_out].
 // scratch: float32 workspace for products cut along K (xr_gemm_tc_scratch_floats bounds what is used); status:
 // device int, set non-zero if a wait gave up.
-XR_EXPORT int xr_gemm_tc(const void* X, const void* W, const float* bias, void* out, int out_dtype, int epilogue, int act, float act_limit,
+// alpha: factor on every sum, ahead of bias and activation (1 for gated products); partial sums carry it.
+XR_EXPORT int xr_gemm_tc(const void* X, const void* W, const float* bias, void* out, int out_dtype, int epilogue, int act, float act_limit, float alpha,
                          int n, int n_out, int K, long long ldx, long long ldo, float* scratch,
                          long long scratch_floats, int* status, int force_splits, int defer_finish, int* splits_used,
                          int w_packed, cudaStream_t stream) {
@@ -817,7 +819,7 @@ XR_EXPORT int xr_gemm_tc(const void* X, const void* W, const float* bias, void* 
     if (out_dtype != XR_F32 && out_dtype != XR_BF16) return XR_ERR_ARG;
     const bool gated = epilogue == TC_EPI_GATED;
     if (act != TC_ACT_NONE && act != TC_ACT_SILU && act != TC_ACT_GELU_TANH && act != TC_ACT_RELU2 && !(act == TC_ACT_SWISH_CLAMP && gated)) return XR_ERR_ARG;
-    if (gated && (!w_packed || bias != nullptr)) return XR_ERR_ARG;
+    if (gated && (!w_packed || bias != nullptr || alpha != 1.0f)) return XR_ERR_ARG;
     const TcPlan pl = plan_product(n, n_out, K, gated, force_splits, defer_finish != 0, scratch ? scratch_floats : 0);
     CUtensorMap mw, mx;
     const int rows_padded = gated ? (int)pl.rows : (n_out + TC_BM - 1) / TC_BM * TC_BM;
@@ -830,6 +832,7 @@ XR_EXPORT int xr_gemm_tc(const void* X, const void* W, const float* bias, void* 
     if (splits_used) *splits_used = splits;
     TcParams p{out, bias, scratch, status, ldo, n, n_out, K, splits, splits > 1 ? TC_EPI_PARTIAL : epilogue, out_dtype,
                act, act_limit, gated ? 1 : 0, pl.bn_eff, w_packed, pl.total_kb, pl.tok_tiles, pl.tok_tiles * ((pl.row_tiles + 1) / 2)};
+    p.alpha = alpha;
     dim3 grid(pl.tok_tiles, pl.row_tiles, splits);
     int rc;
     if (pl.pair) {
@@ -936,7 +939,7 @@ XR_EXPORT int xr_gemm_tc_noalloc(const void* X, const void* W, const float* bias
     // the status word must start at zero; the scratch needs no clearing (every partial that is read was
     // written by this call first)
     if (cudaMemsetAsync(g_noalloc_status_ptr[dev], 0, sizeof(int), stream) != cudaSuccess) return XR_ERR_LAUNCH;
-    int rc = xr_gemm_tc(X, W, bias, out, out_dtype, epilogue, TC_ACT_NONE, 0.f, n, n_out, K, ldx, ldo, g_noalloc_scratch_ptr[dev],
+    int rc = xr_gemm_tc(X, W, bias, out, out_dtype, epilogue, TC_ACT_NONE, 0.f, 1.f, n, n_out, K, ldx, ldo, g_noalloc_scratch_ptr[dev],
                         (long long)XR_NOALLOC_SCRATCH_FLOATS, g_noalloc_status_ptr[dev], want.splits, 0, nullptr, 0, stream);
     if (rc != XR_OK) return rc;
     if (status_out_host != nullptr) {

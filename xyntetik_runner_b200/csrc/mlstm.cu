@@ -286,7 +286,7 @@ k_mlstm_out(const float* __restrict__ o, const TG* __restrict__ proj, long long 
         const float z = xr_to_f32<TG>(g[i]);
         float gate = 1.0f / (1.0f + expf(-z));
         if (gate_silu) gate *= z;
-        dst[i] = xr_from_f32<T>(src[i] * inv * w[(size_t)h * w_head + i] * gate);
+        dst[i] = xr_from_f32<T>(src[i] * inv * (w != nullptr ? w[(size_t)h * w_head + i] : 1.0f) * gate);
     }
 }
 
@@ -339,8 +339,8 @@ XR_EXPORT int xr_mlstm(const void* proj, int dtype, long long ldp, int q_col, in
 }
 
 // The last step alone, for other recurrences: y [n][H * V] (dtype `dtype`) = o / rms(o per head) * w * act(gate), gate [n][ld_gate]
-// (dtype `gate_dtype`: that of y, or float32) from column 0, head h at h * V; w_head: elements between the heads' weights (0: one
-// weight for all heads).
+// (dtype `gate_dtype`: that of y, or float32) from column 0, head h at h * V; w null: no weight; w_head: elements between the heads'
+// weights (0: one weight for all heads).
 XR_EXPORT int xr_head_norm_gate(const float* o, const void* gate, int gate_dtype, long long ld_gate, const float* w, int w_head, int gate_silu,
                                 void* y, int dtype, int n, int H, int V, float eps, cudaStream_t stream) {
     if (n < 1 || H < 1 || V < 1 || w_head < 0) return XR_ERR_ARG;

@@ -2,11 +2,11 @@
 // the experts' products over the rows that chose them, and the weighted sum back into the token's stream.
 //
 //   z = W_router h (float32, a product of the caller);  the `top` largest z are chosen (ties: the lower index),
-//   weights = softmax over the chosen z only;  out[t] += sum_j weight_j * expert_{e_j}(h[t]).
+//   weights = softmax over the chosen z only;  out[t] += scale (sum_j weight_j * expert_{e_j}(h[t]) + sigmoid(g[t]) * shared(h[t])).
 // Other scores, a correction of the choice, groups of experts and a factor on the weights: see k_route_topk and k_route_groups.
 // The router may have more outputs than there are experts: the outputs from E on are identity experts, whose output is h[t]
 // itself.  They take part in the choice, have no rows in the plan (pair_row -1), and the weighted sum adds weight * h[t] for them.
-// An expert is a gated feed-forward: y = gate_act(W_gate h, W_up h), then W_down y (see xr_gate below for the
+// An expert is a feed-forward: y = gate_act(W_gate h, W_up h), or act(W_up h) without a gate, then W_down y (see xr_gate below for the
 // activations).  No step reads anything back to the host: the plan of who computes what is made on the device, and
 // the grids are sized for the worst case (every tile index beyond the plan's count returns at once).
 #include "common.cuh"
@@ -16,14 +16,14 @@
 // Choice: one warp per token.  ids [n][top] int32, wts [n][top] float32 (in the order of descending z).
 // ---------------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(128)
-k_route_topk(const float* __restrict__ z, int* __restrict__ ids, float* __restrict__ wts, int n, int E, int top,
+k_route_topk(const float* __restrict__ z, long long ldz, int* __restrict__ ids, float* __restrict__ wts, int n, int E, int top,
              const float* __restrict__ correction, int sigmoid_scores) {
     xr_pdl_launch();
     xr_pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * 4 + warp;
     if (t >= n) return;
-    const float* row = z + (size_t)t * E;
+    const float* row = z + (size_t)t * ldz;
     float best0 = 0.f, sum = 0.f;
     int last_e = -1;
     float last_v = INFINITY;
@@ -57,12 +57,12 @@ k_route_topk(const float* __restrict__ z, int* __restrict__ ids, float* __restri
     for (int j = 32 + lane; j < top; j += 32) wts[(size_t)t * top + j] /= sum;
 }
 
-// sigmoid_scores: scores s = sigmoid(z); the `top` largest s + correction (correction [E] float32 or null) are chosen and their
+// z: rows of E values, ldz apart.  sigmoid_scores: scores s = sigmoid(z); the `top` largest s + correction (correction [E] float32 or null) are chosen and their
 // weights are s itself, not renormalised.  Otherwise the `top` largest z, weights their softmax.
-XR_EXPORT int xr_route_topk(const float* z, int* ids, float* wts, int n, int E, int top, const float* correction, int sigmoid_scores,
+XR_EXPORT int xr_route_topk(const float* z, long long ldz, int* ids, float* wts, int n, int E, int top, const float* correction, int sigmoid_scores,
                             cudaStream_t stream) {
-    if (n < 1 || E < 1 || top < 1 || top > E || (correction != nullptr && !sigmoid_scores)) return XR_ERR_ARG;
-    xr_launch(k_route_topk, dim3((n + 3) / 4), dim3(128), 0, stream, z, ids, wts, n, E, top, correction, sigmoid_scores ? 1 : 0);
+    if (n < 1 || E < 1 || top < 1 || top > E || ldz < E || (correction != nullptr && !sigmoid_scores)) return XR_ERR_ARG;
+    xr_launch(k_route_topk, dim3((n + 3) / 4), dim3(128), 0, stream, z, ldz, ids, wts, n, E, top, correction, sigmoid_scores ? 1 : 0);
     return xr_launch_status();
 }
 
@@ -240,7 +240,8 @@ XR_EXPORT int xr_moe_gather(const void* h, int dtype, long long ldh, void* out, 
 // the products of the true 32-bit path and of sizes the tensor-core product does not take.
 //  first product (gated = 1): rows gather their token's h (row_src[r] / top); W = [E][2F][K] (an expert's gate rows,
 //    then its up rows); out Y [rows][F] in the activation dtype = gate_act(h . w_gate_f, h . w_up_f).
-//  second product (gated = 0): rows read Y [rows][K = F]; W = [E][N][K]; out Z [rows][N] float32.
+//  first product of experts without a gate (gated = 0, gather = 1): W = [E][F][K]; out Y [rows][F] = act(h . w_f).
+//  second product (gated = 0, gather = 0): rows read Y [rows][K = F]; W = [E][N][K]; out Z [rows][N] float32.
 // Tile: 64 rows x 64 columns (gated: 32 features, gate and up side by side), 256 threads with 4 x 4 results each.
 // ---------------------------------------------------------------------------------------------
 #define MOE_TM 64
@@ -261,7 +262,7 @@ __device__ __forceinline__ float moe_gate(int act, float limit, float g, float u
 template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
 k_moe_gemm(const TA* __restrict__ A, long long lda, const TW* __restrict__ W, TO* __restrict__ out, long long ldo,
-           const int* __restrict__ row_src, const int* __restrict__ tile_group, int top, int N, int K, int gated, int act, float limit) {
+           const int* __restrict__ row_src, const int* __restrict__ tile_group, int top, int N, int K, int gated, int gather, int act, float limit) {
     xr_pdl_launch();
     __shared__ float As[16][64 + 1], Ws[16][64 + 1];
     __shared__ int src_row[64];
@@ -274,7 +275,7 @@ k_moe_gemm(const TA* __restrict__ A, long long lda, const TW* __restrict__ W, TO
     const TW* We = W + (size_t)e * (gated ? 2 : 1) * N * K;
     if (threadIdx.x < 64) {
         const int r = threadIdx.x, s = row_src[r0 + r];
-        src_row[r] = s < 0 ? -1 : (gated ? s / top : r0 + r);
+        src_row[r] = s < 0 ? -1 : (gather ? s / top : r0 + r);
     }
     __syncthreads();
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -320,7 +321,7 @@ k_moe_gemm(const TA* __restrict__ A, long long lda, const TW* __restrict__ W, TO
 #pragma unroll
             for (int j = 0; j < 4; j++) {
                 const int c = c0 + tx + 16 * j;
-                if (c < N) orow[c] = xr_from_f32<TO>(acc[i][j]);
+                if (c < N) orow[c] = xr_from_f32<TO>(moe_gate(act, limit, acc[i][j], 1.0f));
             }
         }
     }
@@ -329,14 +330,14 @@ k_moe_gemm(const TA* __restrict__ A, long long lda, const TW* __restrict__ W, TO
 // a_dtype: of A; w_dtype: of the experts' matrices; max_tiles: tiles of 64 rows the plan may use.
 XR_EXPORT int xr_moe_gemm(const void* A, int a_dtype, long long lda, const void* W, int w_dtype, void* out, int out_dtype,
                           long long ldo, const int* row_src, const int* tile_group, int max_tiles,
-                          int top, int N, int K, int gated, int act, float limit, cudaStream_t stream) {
-    if (max_tiles < 1 || N < 1 || K < 1 || top < 1 || act < 0 || act > 4) return XR_ERR_ARG;
+                          int top, int N, int K, int gated, int gather, int act, float limit, cudaStream_t stream) {
+    if (max_tiles < 1 || N < 1 || K < 1 || top < 1 || act < 0 || act > 4 || (gated && !gather) || (!gated && act == 3)) return XR_ERR_ARG;
     const int cols = gated ? 32 : 64;
     dim3 grid(max_tiles, (N + cols - 1) / cols);
     if (grid.y > 65535) return XR_ERR_ARG;
     typedef __nv_bfloat16 bf;
 #define MG(TA, TW, TO) xr_launch((k_moe_gemm<TA, TW, TO>), grid, dim3(256), 0, stream, (const TA*)A, lda, (const TW*)W, (TO*)out, ldo, \
-                                 row_src, tile_group, top, N, K, gated, act, limit)
+                                 row_src, tile_group, top, N, K, gated, gather, act, limit)
     const int key = a_dtype * 4 + w_dtype * 2 + out_dtype;
     switch (key) {
         case XR_BF16 * 4 + XR_BF16 * 2 + XR_BF16: MG(bf, bf, bf); break;
@@ -352,40 +353,172 @@ XR_EXPORT int xr_moe_gemm(const void* A, int a_dtype, long long lda, const void*
 }
 
 // ---------------------------------------------------------------------------------------------
-// d[t][c] += sum_j wts[t][j] * Z[pair_row[t * top + j]][c], j ascending (float32).  A pair without a row (pair_row -1) is an identity
-// expert's: its term is wts[t][j] * h[t][c].
+// d[t] += scale (sum_j wts[t][j] Z[pair_row[t * top + j]] + sigmoid(sg[t]) sum_s shared[s][t]), j and s ascending (float32).  A pair
+// without a row (pair_row -1) is an identity expert's: its term is wts[t][j] * h[t].  `shared` (null: none): the shared expert's output,
+// or the partial sums of its last product where that was cut along K.  With `nw` the row is then normed in passing:
+// out[t] = d[t] / sqrt(mean(d[t]^2) + eps) * nw.  A block a token; a thread VEC consecutive columns at a time, its first CB_KEEP of
+// them in registers between the two passes.
 // ---------------------------------------------------------------------------------------------
-template <typename T>
-__global__ void __launch_bounds__(256)
-k_moe_combine(float* __restrict__ d, const float* __restrict__ Z, const float* __restrict__ wts, const int* __restrict__ pair_row,
-              const T* __restrict__ h, long long ldh, int n, int width, int top) {
+#define CB_KEEP 4
+
+struct CombineArgs {
+    float* d; const float* Z; const float* wts; const int* pair_row;
+    const void* h; long long ldh;
+    const float* shared; int splits; const float* sg; long long ld_sg;
+    float scale;
+    const float* nw; void* out; float eps;
+    int n, width, top;
+};
+
+template <int VEC> struct CombineVec { float v[VEC]; };
+template <int VEC>
+__device__ __forceinline__ CombineVec<VEC> cb_load(const float* p) {
+    CombineVec<VEC> r;
+    if constexpr (VEC == 4) { const float4 x = xr_ld_now4(reinterpret_cast<const float4*>(p)); r.v[0] = x.x; r.v[1] = x.y; r.v[2] = x.z; r.v[3] = x.w; }
+    else r.v[0] = xr_ld_now(p);
+    return r;
+}
+template <int VEC>
+__device__ __forceinline__ void cb_store(float* p, const CombineVec<VEC>& r) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+    else *p = r.v[0];
+}
+
+template <typename TH, typename TO, int VEC>
+__global__ void __launch_bounds__(1024)
+k_moe_combine(CombineArgs a) {
     xr_pdl_launch();
+    extern __shared__ float cb_sm[];                 // the token's weights [top], then its rows [top]
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, units = a.width / VEC, top = a.top;
+    int* rows = reinterpret_cast<int*>(cb_sm + top);
     xr_pdl_wait();
-    const size_t total = (size_t)n * width;
-    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
-        const size_t t = i / width, c = i % width;
-        float s = 0.f;
-        for (int j = 0; j < top; j++) {
-            const int r = pair_row[t * top + j];
-            float v = 0.f;
-            if (r >= 0) v = Z[(size_t)r * width + c];
-            else if (h != nullptr) v = xr_to_f32<T>(h[t * ldh + c]);
-            s = fmaf(wts[t * top + j], v, s);
+    for (int j = threadIdx.x; j < top; j += blockDim.x) { cb_sm[j] = a.wts[(size_t)t * top + j]; rows[j] = a.pair_row[(size_t)t * top + j]; }
+    __syncthreads();
+    const float gate = a.shared == nullptr ? 0.f : (a.sg == nullptr ? 1.0f : 1.0f / (1.0f + expf(-a.sg[(size_t)t * a.ld_sg])));
+    float* drow = a.d + (size_t)t * a.width;
+    auto value = [&](int u) {
+        const int c = u * VEC;
+        const CombineVec<VEC> old = cb_load<VEC>(drow + c);
+        CombineVec<VEC> s;
+#pragma unroll
+        for (int i = 0; i < VEC; i++) s.v[i] = 0.f;
+        // four rows' loads in flight together (a row that does not exist reads row 0 and counts nothing)
+        for (int j0 = 0; j0 < top; j0 += 4) {
+            CombineVec<VEC> z[4];
+#pragma unroll
+            for (int q = 0; q < 4; q++) {
+                const int j = min(j0 + q, top - 1);
+                z[q] = cb_load<VEC>(a.Z + (size_t)max(rows[j], 0) * a.width + c);
+            }
+#pragma unroll
+            for (int q = 0; q < 4; q++)
+#pragma unroll
+                for (int i = 0; i < VEC; i++) xr_ld_fence(z[q].v[i]);
+#pragma unroll
+            for (int q = 0; q < 4; q++) {
+                if (j0 + q >= top) continue;
+                const bool has = rows[j0 + q] >= 0;
+#pragma unroll
+                for (int i = 0; i < VEC; i++) {
+                    float v = has ? z[q].v[i] : 0.f;
+                    if (!has && a.h != nullptr) v = xr_to_f32<TH>(((const TH*)a.h)[(size_t)t * a.ldh + c + i]);
+                    s.v[i] = fmaf(cb_sm[j0 + q], v, s.v[i]);
+                }
+            }
         }
-        d[i] += s;
+        if (a.shared != nullptr) {
+            float sh[VEC];
+#pragma unroll
+            for (int i = 0; i < VEC; i++) sh[i] = 0.f;
+            for (int s0 = 0; s0 < a.splits; s0 += 4) {
+                CombineVec<VEC> z[4];
+#pragma unroll
+                for (int q = 0; q < 4; q++) z[q] = cb_load<VEC>(a.shared + ((size_t)min(s0 + q, a.splits - 1) * a.n + t) * a.width + c);
+#pragma unroll
+                for (int q = 0; q < 4; q++)
+#pragma unroll
+                    for (int i = 0; i < VEC; i++) xr_ld_fence(z[q].v[i]);
+#pragma unroll
+                for (int q = 0; q < 4; q++)
+#pragma unroll
+                    for (int i = 0; i < VEC; i++) sh[i] += s0 + q < a.splits ? z[q].v[i] : 0.f;
+            }
+#pragma unroll
+            for (int i = 0; i < VEC; i++) s.v[i] = fmaf(gate, sh[i], s.v[i]);
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; i++) s.v[i] = fmaf(a.scale, s.v[i], old.v[i]);
+        cb_store<VEC>(drow + c, s);
+        return s;
+    };
+    CombineVec<VEC> keep[CB_KEEP];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < CB_KEEP; k++) {
+        const int u = threadIdx.x + k * blockDim.x;
+        if (u < units) {
+            keep[k] = value(u);
+#pragma unroll
+            for (int i = 0; i < VEC; i++) ss = fmaf(keep[k].v[i], keep[k].v[i], ss);
+        }
+    }
+    for (int u = threadIdx.x + CB_KEEP * blockDim.x; u < units; u += blockDim.x) {
+        const CombineVec<VEC> v = value(u);
+#pragma unroll
+        for (int i = 0; i < VEC; i++) ss = fmaf(v.v[i], v.v[i], ss);
+    }
+    if (a.nw == nullptr) return;
+    ss = xr_block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)a.width + a.eps);
+    TO* orow = (TO*)a.out + (size_t)t * a.width;
+    auto put = [&](int u, const CombineVec<VEC>& v) {
+        alignas(16) TO w[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; i++) w[i] = xr_from_f32<TO>(v.v[i] * inv * a.nw[u * VEC + i]);
+        if constexpr (VEC == 4) {
+            if constexpr (sizeof(TO) == 4) *reinterpret_cast<float4*>(orow + u * 4) = *reinterpret_cast<float4*>(w);
+            else *reinterpret_cast<uint2*>(orow + u * 4) = *reinterpret_cast<uint2*>(w);
+        } else orow[u] = w[0];
+    };
+#pragma unroll
+    for (int k = 0; k < CB_KEEP; k++) {
+        const int u = threadIdx.x + k * blockDim.x;
+        if (u < units) put(u, keep[k]);
+    }
+    for (int u = threadIdx.x + CB_KEEP * blockDim.x; u < units; u += blockDim.x) {         // (this thread's own stores)
+        CombineVec<VEC> v;
+#pragma unroll
+        for (int i = 0; i < VEC; i++) v.v[i] = drow[u * VEC + i];
+        put(u, v);
     }
 }
 
-// h [n][ldh] in h_dtype: what the experts read, for identity experts; null: there are none.
-XR_EXPORT int xr_moe_combine(float* d, const float* Z, const float* wts, const int* pair_row, const void* h, int h_dtype, long long ldh, int n,
-                             int width, int top, cudaStream_t stream) {
-    if (n < 1 || width < 1 || top < 1 || (h != nullptr && ldh < width)) return XR_ERR_ARG;
-    const size_t total = (size_t)n * width;
-    int blocks = (int)((total + 255) / 256 < (size_t)xr_sm_count() * 16 ? (total + 255) / 256 : xr_sm_count() * 16);
-    if (h == nullptr || h_dtype == XR_F32)
-        xr_launch((k_moe_combine<float>), dim3(blocks), dim3(256), 0, stream, d, Z, wts, pair_row, (const float*)h, ldh, n, width, top);
-    else if (h_dtype == XR_BF16)
-        xr_launch((k_moe_combine<__nv_bfloat16>), dim3(blocks), dim3(256), 0, stream, d, Z, wts, pair_row, (const __nv_bfloat16*)h, ldh, n, width, top);
-    else return XR_ERR_ARG;
+// d [n][width] float32.  h [n][ldh] in h_dtype: what the experts read, for identity experts; null: there are none.  shared
+// [splits][n][width] float32 with sg (n values, ld_sg apart; null: no gate); nw [width] with out [n][width] in out_dtype.
+XR_EXPORT int xr_moe_combine(float* d, const float* Z, const float* wts, const int* pair_row, const void* h, int h_dtype, long long ldh,
+                             const float* shared, int splits, const float* sg, long long ld_sg, float scale, const float* nw, void* out,
+                             int out_dtype, float eps, int n, int width, int top, cudaStream_t stream) {
+    if (n < 1 || width < 1 || top < 1 || top > 4096 || (h != nullptr && ldh < width) || (shared != nullptr && splits < 1) || (nw == nullptr) != (out == nullptr))
+        return XR_ERR_ARG;
+    if ((h != nullptr && h_dtype != XR_F32 && h_dtype != XR_BF16) || (out != nullptr && out_dtype != XR_F32 && out_dtype != XR_BF16)) return XR_ERR_ARG;
+    CombineArgs a{d, Z, wts, pair_row, h, ldh, shared, splits, sg, ld_sg, scale, nw, out, eps, n, width, top};
+    const bool vec = !(width & 3) && !(((uintptr_t)d | (uintptr_t)Z | (uintptr_t)shared | (uintptr_t)out) & 15);
+    // (few tokens: nothing but a row's own threads hides its loads' latency)
+    const int units = vec ? width / 4 : width, most = n <= xr_sm_count() ? 1024 : 256, threads = units >= most ? most : (units + 31) / 32 * 32;
+    const size_t smem = (size_t)top * 8;
+#define CB1(TH, TO, VEC) xr_launch((k_moe_combine<TH, TO, VEC>), dim3(n), dim3(threads), smem, stream, a)
+#define CB(TH, TO)                                                                                                                           \
+    do {                                                                                                                                     \
+        if (vec) CB1(TH, TO, 4);                                                                                                             \
+        else CB1(TH, TO, 1);                                                                                                                 \
+    } while (0)
+    const bool hb = h != nullptr && h_dtype == XR_BF16, ob = out != nullptr && out_dtype == XR_BF16;
+    if (hb && ob) CB(__nv_bfloat16, __nv_bfloat16);
+    else if (hb) CB(__nv_bfloat16, float);
+    else if (ob) CB(float, __nv_bfloat16);
+    else CB(float, float);
+#undef CB
+#undef CB1
     return xr_launch_status();
 }

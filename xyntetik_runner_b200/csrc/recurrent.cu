@@ -1,4 +1,4 @@
-// Three linear recurrences with a fixed-size float32 state per request slot.
+// Linear recurrences with a fixed-size float32 state per request slot.
 //
 // (1) The real-gated linear recurrent unit (the recurrence of Griffin's recurrent block).  With R channels in B blocks of
 //     R / B, a short causal convolution per channel, and per token the projections' rows y' and x' (float32, biases included):
@@ -13,8 +13,11 @@
 //     portion's tokens, the read-out times the gated branch, and the slot's new tail.
 //
 // (2) Linear attention with a constant decay per head ("lightning attention"): S [D][V] per head,
-//       S <- decay_h S + k v^T,   o = S^T q,   q, k, v the projections' rows behind their activation.
+//       S <- decay_h S + k v^T,   o = c S^T q,   q, k, v the projections' rows, behind an activation or as they are, c a constant.
 //     k_decay_scan, a warp per eight value columns of a head: the state in registers, see there.
+//     With a decay per key channel and token ("gated linear attention"), S <- diag(a_t) S + k v^T:
+//       a_t = sigmoid(A2 (A1 h_t) + b)^(1/tau),   A1 h_t of a few values a token, columns of the same projection.
+//     k_key_decay makes the rows a [n][H D]; the walk takes them beside q, k and v.
 //
 // (3) The state-space dual recurrence of Mamba-2: S [N][V] per head, head h reading key and query rows B, C of group h / (H / G),
 //       S <- exp(-exp(A_log_h) dt) S + dt B x^T,   y = S^T C + D_h x,   dt = softplus(dt' + dt_bias_h)
@@ -310,10 +313,14 @@ XR_EXPORT int xr_rglru(float* proj, long long ldp, int y_col, int x_col, const f
 // registers before this chunk is walked and stored behind it (16 bytes a load where sizes and addresses allow: VEC).  A step of
 // many tokens applies silu to the rows beforehand, in
 // place (k_silu_cols); a step of few applies it on the way into shared memory.
-// SSD: the decay and the factor on the value come per token and head (coef), heads share key and query rows by `rep`, the
+// KIND: DS_HEAD: a constant decay per head.  DS_KEY: a decay per key channel and token, rows [n][H D] of their own.
+// DS_SSD: the decay and the factor on the value come per token and head (coef), heads share key and query rows by `rep`, the
 // value times skip[h] joins the read-out, a column's state lies together in memory ([H][V][D] instead of [H][D][V]), and the
 // blocks of a portion leave the convolution's new tail behind the walk.
 #define DA_WARPS 8
+#define DS_HEAD 0
+#define DS_SSD 1
+#define DS_KEY 2
 
 struct SsdArgs {
     const float* coef;           // [n][H][2]: decay, dt
@@ -321,6 +328,10 @@ struct SsdArgs {
     const float* raw;            // the convolution's inputs, row stride ld_raw, CH columns
     long long ld_raw;
     int CH, taps, rep;
+};
+struct KeyDecayArgs {
+    const float* rows;           // [n][H D]: the decays
+    float read_scale;            // factor on the read-outs (DS_HEAD too)
 };
 
 __global__ void k_silu_cols(float* __restrict__ rows, long long ld, int cols, size_t total) {
@@ -332,22 +343,24 @@ __global__ void k_silu_cols(float* __restrict__ rows, long long ld, int cols, si
     }
 }
 
-template <int JD, int VC, int CH, bool VEC, bool SSD>
+template <int JD, int VC, int CH, bool VEC, int KIND>
 __global__ void __launch_bounds__(32 * DA_WARPS)
 k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col, int v_col, const float* __restrict__ decay,
              float* __restrict__ state, long long state_stride, const int* __restrict__ seg_start, const int* __restrict__ seg_len,
-             const int* __restrict__ seg_slot, float* __restrict__ o, int H, int D, int V, int activated, SsdArgs ssd) {
+             const int* __restrict__ seg_slot, float* __restrict__ o, int H, int D, int V, int activated, SsdArgs ssd, KeyDecayArgs key) {
     xr_pdl_launch();
-    constexpr int COLS = VC * DA_WARPS, DP = 32 * JD, RW = 2 * DP + COLS, TB = 32 / VC;
+    constexpr bool SSD = KIND == DS_SSD, KEY = KIND == DS_KEY;
+    // a token's row in shared memory: q [DP], k [DP] (zeros behind D), DS_KEY: its decays [DP], the block's v [COLS]
+    constexpr int COLS = VC * DA_WARPS, DP = 32 * JD, VA = (KEY ? 3 : 2) * DP, RW = VA + COLS, TB = 32 / VC;
     constexpr int PER = (CH * RW + 32 * DA_WARPS - 1) / (32 * DA_WARPS);
     static_assert(CH % TB == 0, "a chunk is whole batches of tokens");
-    __shared__ __align__(16) float da_sm[2 * CH * RW];       // a token's row: q [DP], k [DP] (zeros behind D), the block's v [COLS]
+    extern __shared__ __align__(16) float da_sm[];           // two chunks of CH rows
     __shared__ __align__(8) float da_coef[SSD ? 2 * CH * 2 : 2];       // SSD: a token's decay and dt
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int vb = blockIdx.x * COLS, v0 = vb + warp * VC, h = blockIdx.y, seg = blockIdx.z;
     const int start = seg_start[seg], len = seg_len[seg];
     const int g = SSD ? h / ssd.rep : h;                     // the head of the query and key rows
-    const float dec = SSD ? 0.f : decay[h], skip = SSD ? ssd.skip[h] : 0.f;
+    const float dec = KIND == DS_HEAD ? decay[h] : 0.f, skip = SSD ? ssd.skip[h] : 0.f;
     float* slot = state + (size_t)seg_slot[seg] * state_stride;
     float* st = slot + (size_t)h * D * V;
     auto at = [&](int d, int c) -> size_t { return SSD ? (size_t)(v0 + c) * D + d : (size_t)d * V + v0 + c; };
@@ -400,7 +413,8 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
                     const float* row = proj + (size_t)(start + i) * ldp;
                     if (cc < DP) { if (cc < D) v = xr_ld_now4(reinterpret_cast<const float4*>(row + q_col + g * D + cc)); }
                     else if (cc < 2 * DP) { if (cc - DP < D) v = xr_ld_now4(reinterpret_cast<const float4*>(row + k_col + g * D + cc - DP)); }
-                    else if (vb + cc - 2 * DP < V) v = xr_ld_now4(reinterpret_cast<const float4*>(row + v_col + h * V + vb + cc - 2 * DP));
+                    else if (KEY && cc < VA) { if (cc - 2 * DP < D) v = xr_ld_now4(reinterpret_cast<const float4*>(key.rows + ((size_t)(start + i) * H + h) * D + cc - 2 * DP)); }
+                    else if (vb + cc - VA < V) v = xr_ld_now4(reinterpret_cast<const float4*>(row + v_col + h * V + vb + cc - VA));
                 }
                 stage4[k] = v;
             }
@@ -416,7 +430,8 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
                     const float* row = proj + (size_t)(start + i) * ldp;
                     if (cc < DP) { if (cc < D) v = xr_ld_now(row + q_col + g * D + cc); }
                     else if (cc < 2 * DP) { if (cc - DP < D) v = xr_ld_now(row + k_col + g * D + cc - DP); }
-                    else if (vb + cc - 2 * DP < V) v = xr_ld_now(row + v_col + h * V + vb + cc - 2 * DP);
+                    else if (KEY && cc < VA) { if (cc - 2 * DP < D) v = xr_ld_now(key.rows + ((size_t)(start + i) * H + h) * D + cc - 2 * DP); }
+                    else if (vb + cc - VA < V) v = xr_ld_now(row + v_col + h * V + vb + cc - VA);
                 }
                 stage[k] = v;
             }
@@ -456,7 +471,7 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
             for (int k = 0; k < TB * VC; k++) acc[k] = 0.f;
             auto token = [&](int tb) {
                 const float* row = base + (t0 + tb) * RW;
-                float q[JD], k[JD], v[VC];
+                float q[JD], k[JD], v[VC], ak[KEY ? JD : 1];
                 float a = dec;
                 if constexpr (JD % 4 == 0) {
 #pragma unroll
@@ -465,24 +480,35 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
                         const float4 b = *reinterpret_cast<const float4*>(row + DP + lane * JD + j);
                         q[j] = a.x; q[j + 1] = a.y; q[j + 2] = a.z; q[j + 3] = a.w;
                         k[j] = b.x; k[j + 1] = b.y; k[j + 2] = b.z; k[j + 3] = b.w;
+                        if constexpr (KEY) {
+                            const float4 c = *reinterpret_cast<const float4*>(row + 2 * DP + lane * JD + j);
+                            ak[j] = c.x; ak[j + 1] = c.y; ak[j + 2] = c.z; ak[j + 3] = c.w;
+                        }
                     }
                 } else if constexpr (JD == 2) {
                     const float2 a = *reinterpret_cast<const float2*>(row + lane * 2);
                     const float2 b = *reinterpret_cast<const float2*>(row + DP + lane * 2);
                     q[0] = a.x; q[1] = a.y; k[0] = b.x; k[1] = b.y;
+                    if constexpr (KEY) {
+                        const float2 c = *reinterpret_cast<const float2*>(row + 2 * DP + lane * 2);
+                        ak[0] = c.x; ak[1] = c.y;
+                    }
                 } else {
 #pragma unroll
-                    for (int j = 0; j < JD; j++) { q[j] = row[lane * JD + j]; k[j] = row[DP + lane * JD + j]; }
+                    for (int j = 0; j < JD; j++) {
+                        q[j] = row[lane * JD + j]; k[j] = row[DP + lane * JD + j];
+                        if constexpr (KEY) ak[j] = row[2 * DP + lane * JD + j];
+                    }
                 }
                 if constexpr (VC % 4 == 0) {
 #pragma unroll
                     for (int c = 0; c < VC; c += 4) {
-                        const float4 a = *reinterpret_cast<const float4*>(row + 2 * DP + warp * VC + c);
+                        const float4 a = *reinterpret_cast<const float4*>(row + VA + warp * VC + c);
                         v[c] = a.x; v[c + 1] = a.y; v[c + 2] = a.z; v[c + 3] = a.w;
                     }
                 } else {
 #pragma unroll
-                    for (int c = 0; c < VC; c++) v[c] = row[2 * DP + warp * VC + c];
+                    for (int c = 0; c < VC; c++) v[c] = row[VA + warp * VC + c];
                 }
                 if constexpr (SSD) {
                     const float2 ad = *reinterpret_cast<const float2*>(da_coef + ((ch & 1) * CH + t0 + tb) * 2);
@@ -494,7 +520,7 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
                 for (int j = 0; j < JD; j++) {
 #pragma unroll
                     for (int c = 0; c < VC; c++) {
-                        s[c][j] = fmaf(a, s[c][j], k[j] * v[c]);
+                        s[c][j] = fmaf(KEY ? ak[KEY ? j : 0] : a, s[c][j], k[j] * v[c]);
                         acc[tb * VC + c] = fmaf(s[c][j], q[j], acc[tb * VC + c]);
                     }
                 }
@@ -524,7 +550,8 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
             const int tb = mine / VC, c = mine % VC;
             if (t0 + tb < here && v0 + c < V) {
                 float y = acc[0];
-                if constexpr (SSD) y = fmaf(skip, base[(t0 + tb) * RW + 2 * DP + warp * VC + c], y);
+                if constexpr (SSD) y = fmaf(skip, base[(t0 + tb) * RW + VA + warp * VC + c], y);
+                else y *= key.read_scale;
                 o[(size_t)(start + ch * CH + t0 + tb) * H * V + (size_t)h * V + v0 + c] = y;
             }
         }
@@ -558,31 +585,29 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
                                   blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
 }
 
-// proj [n][ldp] float32: pre-activations of q at q_col [H][D], k at k_col [H][D], v at v_col [H][V] (`cols` columns from the first
-// of them to the last of v, which a step of many tokens activates in place); decay [H] float32; state [slots][state_stride]
-// float32, S [H][D][V];  o [n][H V] float32 receives the read-outs.
-XR_EXPORT int xr_decay_attention(float* proj, long long ldp, int q_col, int k_col, int v_col, const float* decay, float* state,
-                                 long long state_stride, const int* seg_start, const int* seg_len, const int* seg_slot, float* o, int n, int n_seg,
-                                 int H, int D, int V, cudaStream_t stream) {
-    if (n < 1 || n_seg < 1 || H < 1 || D < 1 || V < 1 || D > 256 || n_seg > 65535 || H > 65535 || state_stride < (long long)H * D * V)
-        return XR_ERR_ARG;
-    // q, k, v lie side by side from q_col on (the caller's layout): one pass activates them all
-    const bool many = n > 16 && k_col == q_col + H * D && v_col == k_col + H * D;
-    if (many) {
-        const size_t total = (size_t)n * (2 * H * D + H * V);
-        const int blocks = (int)((total + 255) / 256 < (size_t)xr_sm_count() * 16 ? (total + 255) / 256 : xr_sm_count() * 16);
-        xr_launch(k_silu_cols, dim3(blocks), dim3(256), 0, stream, proj + q_col, ldp, 2 * H * D + H * V, total);
-    }
+// bytes of shared memory a block of the walk takes: two chunks of CH tokens' rows
+static constexpr size_t decay_scan_smem(int JD, int VC, int CH, int KIND) {
+    return (size_t)2 * CH * ((KIND == DS_KEY ? 3 : 2) * 32 * JD + VC * DA_WARPS) * sizeof(float);
+}
+
+template <int KIND>
+static int launch_decay_scan(const float* proj, long long ldp, int q_col, int k_col, int v_col, const float* decay, float* state, long long state_stride,
+                             const int* seg_start, const int* seg_len, const int* seg_slot, float* o, int n, int n_seg, int H, int D, int V, bool ready,
+                             KeyDecayArgs key, cudaStream_t stream) {
     // (a step with long portions is a few long-lived blocks: they start behind the kernel ahead, not into its last wave)
     const bool walk = n > 4 * n_seg;
     // 16 bytes a load where every row, column offset and size falls on a 16-byte border
-    const bool vec = !((D | V | ldp | q_col | k_col | v_col) & 3) && !((uintptr_t)proj & 15);
-#define DS_ARGS(JD, VC, CH) dim3((V + VC * DA_WARPS - 1) / (VC * DA_WARPS), H, n_seg), dim3(32 * DA_WARPS), 0, stream,                      \
-                            (const float*)proj, ldp, q_col, k_col, v_col, decay, state, state_stride, seg_start, seg_len, seg_slot, o, H, D, V, many ? 1 : 0, SsdArgs{}
+    const bool vec = !((D | V | ldp | q_col | k_col | v_col) & 3) && !(((uintptr_t)proj | (uintptr_t)key.rows) & 15);
+#define DS_ARGS(JD, VC, CH) dim3((V + VC * DA_WARPS - 1) / (VC * DA_WARPS), H, n_seg), dim3(32 * DA_WARPS), decay_scan_smem(JD, VC, CH, KIND), stream, \
+                            proj, ldp, q_col, k_col, v_col, decay, state, state_stride, seg_start, seg_len, seg_slot, o, H, D, V, ready ? 1 : 0, SsdArgs{}, key
 #define DS1(JD, VC, CH, VEC)                                                                                                                 \
     do {                                                                                                                                     \
-        if (walk) xr_launch_behind((k_decay_scan<JD, VC, CH, VEC, false>), DS_ARGS(JD, VC, CH));                                                    \
-        else xr_launch((k_decay_scan<JD, VC, CH, VEC, false>), DS_ARGS(JD, VC, CH));                                                                \
+        if (decay_scan_smem(JD, VC, CH, KIND) > 48 * 1024 &&                                                                                 \
+            cudaFuncSetAttribute(k_decay_scan<JD, VC, CH, VEC, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize,                           \
+                                 (int)decay_scan_smem(JD, VC, CH, KIND)) != cudaSuccess)                                                     \
+            return XR_ERR_LAUNCH;                                                                                                            \
+        if (walk) xr_launch_behind((k_decay_scan<JD, VC, CH, VEC, KIND>), DS_ARGS(JD, VC, CH));                                              \
+        else xr_launch((k_decay_scan<JD, VC, CH, VEC, KIND>), DS_ARGS(JD, VC, CH));                                                          \
     } while (0)
 #define DS(JD, VC, CH)                                                                                                                       \
     do {                                                                                                                                     \
@@ -597,6 +622,79 @@ XR_EXPORT int xr_decay_attention(float* proj, long long ldp, int q_col, int k_co
 #undef DS1
 #undef DS_ARGS
     return xr_launch_status();
+}
+
+// proj [n][ldp] float32: q at q_col [H][D], k at k_col [H][D], v at v_col [H][V]; with `silu` their pre-activations (columns from the
+// first of q to the last of v, which a step of many tokens activates in place), else as they are; decay [H] float32; state
+// [slots][state_stride] float32, S [H][D][V];  o [n][H V] float32 receives the read-outs, times read_scale.
+XR_EXPORT int xr_decay_attention(float* proj, long long ldp, int q_col, int k_col, int v_col, const float* decay, float* state,
+                                 long long state_stride, const int* seg_start, const int* seg_len, const int* seg_slot, float* o, int n, int n_seg,
+                                 int H, int D, int V, int silu, float read_scale, cudaStream_t stream) {
+    if (n < 1 || n_seg < 1 || H < 1 || D < 1 || V < 1 || D > 256 || n_seg > 65535 || H > 65535 || state_stride < (long long)H * D * V)
+        return XR_ERR_ARG;
+    // q, k, v lie side by side from q_col on (the caller's layout): one pass activates them all
+    const bool many = silu && n > 16 && k_col == q_col + H * D && v_col == k_col + H * D;
+    if (many) {
+        const size_t total = (size_t)n * (2 * H * D + H * V);
+        const int blocks = (int)((total + 255) / 256 < (size_t)xr_sm_count() * 16 ? (total + 255) / 256 : xr_sm_count() * 16);
+        xr_launch(k_silu_cols, dim3(blocks), dim3(256), 0, stream, proj + q_col, ldp, 2 * H * D + H * V, total);
+    }
+    return launch_decay_scan<DS_HEAD>(proj, ldp, q_col, k_col, v_col, decay, state, state_stride, seg_start, seg_len, seg_slot, o, n, n_seg, H, D, V,
+                                      many || !silu, KeyDecayArgs{nullptr, read_scale}, stream);
+}
+
+// ---------------------------------------------------------------------------------------------
+// Decays per key channel: out[t][c] = sigmoid(z)^(1/tau) = exp(log sigmoid(z) / tau), z = bias[c] + sum_r w_t[r][c] in[t][r]; `in` R
+// columns of a wider float32 row, w_t the matrix transposed ([R][C], so that a warp reads a row).  A thread a channel with KD_T
+// tokens' sums; the tokens' rows lie in shared memory, R of them at a time.
+// ---------------------------------------------------------------------------------------------
+#define KD_R 64
+template <int KD_T>
+__global__ void __launch_bounds__(128)
+k_key_decay(const float* __restrict__ in, long long ld_in, const float* __restrict__ w_t, const float* __restrict__ bias, float* __restrict__ out,
+            int n, int R, int C, float inv_tau, int early) {
+    if (early) xr_pdl_launch();                  // (a walk of long portions stays behind this kernel: see xr_launch_behind)
+    __shared__ float rows[KD_R][KD_T];
+    const int c = blockIdx.x * 128 + threadIdx.x, t0 = blockIdx.y * KD_T, cc = min(c, C - 1);
+    float z[KD_T];
+    const float b = bias[cc];
+#pragma unroll
+    for (int i = 0; i < KD_T; i++) z[i] = b;
+    xr_pdl_wait();
+    for (int r0 = 0; r0 < R; r0 += KD_R) {
+        const int rn = min(KD_R, R - r0);
+        for (int e = threadIdx.x; e < rn * KD_T; e += 128) {
+            const int t = t0 + e / rn, r = e % rn;
+            rows[r][e / rn] = t < n ? in[(size_t)t * ld_in + r0 + r] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll 8
+        for (int r = 0; r < rn; r++) {
+            const float w = w_t[(size_t)(r0 + r) * C + cc];
+#pragma unroll
+            for (int i = 0; i < KD_T; i++) z[i] = fmaf(w, rows[r][i], z[i]);
+        }
+        __syncthreads();
+    }
+    if (c >= C) return;
+#pragma unroll
+    for (int i = 0; i < KD_T; i++)
+        if (t0 + i < n) out[(size_t)(t0 + i) * C + c] = expf((fminf(z[i], 0.f) - log1pf(expf(-fabsf(z[i])))) * inv_tau);
+}
+
+// Linear attention with a decay per key channel: q, k, v as in xr_decay_attention without an activation; the decays' inner values at
+// a_col (R columns of proj), w_t [R][H D], bias [H D] float32; decays [n][H D] float32 scratch.
+XR_EXPORT int xr_key_decay_attention(const float* proj, long long ldp, int q_col, int k_col, int v_col, int a_col, const float* w_t, const float* bias,
+                                     int R, float tau, float* decays, float* state, long long state_stride, const int* seg_start, const int* seg_len,
+                                     const int* seg_slot, float* o, int n, int n_seg, int H, int D, int V, float read_scale, cudaStream_t stream) {
+    if (n < 1 || n_seg < 1 || H < 1 || D < 1 || V < 1 || D > 256 || R < 1 || !(tau > 0.f) || n_seg > 65535 || H > 65535 || n > 65535 * 4 ||
+        state_stride < (long long)H * D * V)
+        return XR_ERR_ARG;
+    const int C = H * D, early = n > 4 * n_seg ? 0 : 1;
+    if (n > 64) xr_launch((k_key_decay<16>), dim3((C + 127) / 128, (n + 15) / 16), dim3(128), 0, stream, proj + a_col, ldp, w_t, bias, decays, n, R, C, 1.0f / tau, early);
+    else xr_launch((k_key_decay<4>), dim3((C + 127) / 128, (n + 3) / 4), dim3(128), 0, stream, proj + a_col, ldp, w_t, bias, decays, n, R, C, 1.0f / tau, early);
+    return launch_decay_scan<DS_KEY>(proj, ldp, q_col, k_col, v_col, nullptr, state, state_stride, seg_start, seg_len, seg_slot, o, n, n_seg, H, D, V,
+                                     true, KeyDecayArgs{decays, read_scale}, stream);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -678,12 +776,12 @@ XR_EXPORT int xr_ssd(const float* proj, long long ldp, int x_col, int dt_col, co
     const bool walk = n > 4 * n_seg;
     const bool vec = !((N | V) & 3) && !((uintptr_t)xbc & 15);
     const SsdArgs ssd{coef, skip, proj + x_col, ldp, CH, taps, H / G};
-#define SS_ARGS(VC) dim3((V + VC * DA_WARPS - 1) / (VC * DA_WARPS), H, n_seg), dim3(32 * DA_WARPS), 0, stream, (const float*)xbc, (long long)CH,            \
-                    H * V + G * N, H * V, 0, (const float*)nullptr, state, state_stride, seg_start, seg_len, seg_slot, y, H, N, V, 1, ssd
+#define SS_ARGS(JD, VC, CK) dim3((V + VC * DA_WARPS - 1) / (VC * DA_WARPS), H, n_seg), dim3(32 * DA_WARPS), decay_scan_smem(JD, VC, CK, DS_SSD), stream, (const float*)xbc, (long long)CH,            \
+                    H * V + G * N, H * V, 0, (const float*)nullptr, state, state_stride, seg_start, seg_len, seg_slot, y, H, N, V, 1, ssd, KeyDecayArgs{nullptr, 1.0f}
 #define SS1(JD, VC, CK, VEC)                                                                                                                 \
     do {                                                                                                                                     \
-        if (walk) xr_launch_behind((k_decay_scan<JD, VC, CK, VEC, true>), SS_ARGS(VC));                                                      \
-        else xr_launch((k_decay_scan<JD, VC, CK, VEC, true>), SS_ARGS(VC));                                                                  \
+        if (walk) xr_launch_behind((k_decay_scan<JD, VC, CK, VEC, DS_SSD>), SS_ARGS(JD, VC, CK));                                                      \
+        else xr_launch((k_decay_scan<JD, VC, CK, VEC, DS_SSD>), SS_ARGS(JD, VC, CK));                                                                  \
     } while (0)
 #define SS(JD, VC, CK)                                                                                                                       \
     do {                                                                                                                                     \

@@ -52,9 +52,9 @@ def _declare(L: ctypes.CDLL) -> None:
         "xr_rope_store": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _ll, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
         "xr_act_mul": [_vp, _vp, _i, _i, _i, _i, _i, _f, _vp],
         "xr_residual_add": [_vp, _vp, _i, _i, _i, _vp],
-        "xr_gemm_simt": [_vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _ll, _ll, _vp],
+        "xr_gemm_simt": [_vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _ll, _ll, _f, _vp],
         "xr_attention_simt": [_vp, _vp, _i, _vp, _vp, _vp, _vp, _ll, _ll, _ll, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _f, _i, _vp, _i, _vp],
-        "xr_gemm_tc": [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _i, _ll, _ll, _vp, _ll, _vp, _i, _i, ctypes.POINTER(ctypes.c_int), _i, _vp],
+        "xr_gemm_tc": [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _f, _i, _i, _i, _ll, _ll, _vp, _ll, _vp, _i, _i, ctypes.POINTER(ctypes.c_int), _i, _vp],
         "xr_finish_add_rmsnorm": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _vp],
         "xr_finish_plain": [_vp, _i, _vp, _vp, _i, _i, _i, _i, _ll, _vp],
         "xr_finish_rope_store": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
@@ -87,14 +87,14 @@ def _declare(L: ctypes.CDLL) -> None:
         "xr_delta": [_vp, _i, _ll, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
         "xr_head_norm_gate": [_vp, _vp, _i, _ll, _vp, _i, _i, _vp, _i, _i, _i, _i, _f, _vp],
         "xr_mlstm": [_vp, _i, _ll, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _f, _vp],
-        "xr_route_topk": [_vp, _vp, _vp, _i, _i, _i, _vp, _i, _vp],
+        "xr_route_topk": [_vp, _ll, _vp, _vp, _i, _i, _i, _vp, _i, _vp],
         "xr_moe_plan": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
         "xr_moe_gather": [_vp, _i, _ll, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
         "xr_gemm_tc_grouped": [_vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _i, _ll, _ll, _i, _vp, _i, _vp, _vp],
         "xr_moe_tile_rows": [],
-        "xr_moe_gemm": [_vp, _i, _ll, _vp, _i, _vp, _i, _ll, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _vp],
+        "xr_moe_gemm": [_vp, _i, _ll, _vp, _i, _vp, _i, _ll, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
         "xr_route_groups": [_vp, _vp, _vp, _i, _i, _i, _vp, _i, _i, _f, _vp],
-        "xr_moe_combine": [_vp, _vp, _vp, _vp, _vp, _i, _ll, _i, _i, _i, _vp],
+        "xr_moe_combine": [_vp, _vp, _vp, _vp, _vp, _i, _ll, _vp, _i, _vp, _ll, _f, _vp, _vp, _i, _f, _i, _i, _i, _vp],
         "xr_embed_pair": [_vp, _vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _ll, _vp],
         "xr_last_token": [_vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _vp],
         "xr_norm_add": [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp, _vp, _i, _vp],
@@ -106,7 +106,8 @@ def _declare(L: ctypes.CDLL) -> None:
         "xr_row_norm_gate": [_vp, _vp, _ll, _vp, _vp, _i, _i, _i, _f, _f, _vp],
         "xr_ssd": [_vp, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
         "xr_silu_gate_norm": [_vp, _vp, _ll, _vp, _vp, _i, _i, _i, _i, _f, _vp],
-        "xr_decay_attention": [_vp, _ll, _i, _i, _i, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+        "xr_decay_attention": [_vp, _ll, _i, _i, _i, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _vp],
+        "xr_key_decay_attention": [_vp, _ll, _i, _i, _i, _i, _vp, _vp, _i, _f, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _vp],
     }
     for name, args in sig.items():
         fn = getattr(L, name)
@@ -285,8 +286,8 @@ def residual_add(x: torch.Tensor, delta: torch.Tensor) -> None:
 
 
 def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
-              accumulate: bool = False) -> None:
-    """out[t][r] (+)= sum_k x[t][k] w[r][k] (+ bias[r]) in float32 FMA.  Rows of x and out may be strided."""
+              accumulate: bool = False, alpha: float = 1.0) -> None:
+    """out[t][r] (+)= alpha sum_k x[t][k] w[r][k] (+ bias[r]) in float32 FMA.  Rows of x and out may be strided."""
     for t in (x, w, out, bias):
         if t is not None and not t.is_cuda:
             raise KernelError("kernel arguments must be CUDA tensors")
@@ -297,7 +298,7 @@ def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optiona
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == n_out)
     _check(lib().xr_gemm_simt(x.data_ptr(), dtype_code(x.dtype), w.data_ptr(), dtype_code(w.dtype), _ptr(bias),
                               out.data_ptr(), dtype_code(out.dtype), int(accumulate), n, n_out, k,
-                              x.stride(0), out.stride(0), _stream()), "gemm_simt")
+                              x.stride(0), out.stride(0), float(alpha), _stream()), "gemm_simt")
     _count()
 
 
@@ -527,7 +528,7 @@ _SPLITS_USED = ctypes.c_int(1)           # where xr_gemm_tc says how it cut the 
 _SPLITS_USED_REF = ctypes.byref(_SPLITS_USED)
 
 
-def _gemm_tc(x, w, out, bias, epilogue, act, force_splits, defer, packed_rows, act_limit=0.0):
+def _gemm_tc(x, w, out, bias, epilogue, act, force_splits, defer, packed_rows, act_limit=0.0, alpha=1.0):
     n, k = x.shape
     gated = epilogue == EPI_GATED
     if packed_rows is not None:
@@ -545,7 +546,7 @@ def _gemm_tc(x, w, out, bias, epilogue, act, force_splits, defer, packed_rows, a
     assert not defer or not gated
     ws = workspace(x.device)
     at, room = ws.room()
-    _check(lib().xr_gemm_tc(x.data_ptr(), w.data_ptr(), _ptr(bias), out.data_ptr(), dtype_code(out.dtype), epilogue, int(act), float(act_limit),
+    _check(lib().xr_gemm_tc(x.data_ptr(), w.data_ptr(), _ptr(bias), out.data_ptr(), dtype_code(out.dtype), epilogue, int(act), float(act_limit), float(alpha),
                             n, n_out, k, x.stride(0), out.stride(0), at, room,
                             ws.status_ptr, force_splits, int(defer), _SPLITS_USED_REF,
                             int(packed_rows is not None), _stream()), "gemm_tc")
@@ -559,21 +560,22 @@ def _gemm_tc(x, w, out, bias, epilogue, act, force_splits, defer, packed_rows, a
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
             epilogue: int = EPI_STORE, force_splits: int = 0, packed_rows: Optional[int] = None, act: Optional[int] = None,
-            act_limit: float = 0.0) -> int:
-    """bfloat16 product on tcgen05.  EPI_STORE: out[t][r] = act(x.w + bias); EPI_ADD: float32 out += x.w + bias;
+            act_limit: float = 0.0, alpha: float = 1.0) -> int:
+    """bfloat16 product on tcgen05.  EPI_STORE: out[t][r] = act(alpha x.w + bias); EPI_ADD: float32 out += alpha x.w + bias;
     EPI_GATED: w from ``pack_weight(w, halves=2)``, out[t][f] = act(x.w_gate[f]) * (x.w_up[f]) (act defaults to SiLU).
     Returns the number of K splits used."""
     if act is None:
         act = ACT_SILU if epilogue == EPI_GATED else ACT_NONE
-    return _gemm_tc(x, w, out, bias, epilogue, act, force_splits, False, packed_rows, act_limit)
+    return _gemm_tc(x, w, out, bias, epilogue, act, force_splits, False, packed_rows, act_limit, alpha)
 
 
 def gemm_tc_deferred(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
-                     epilogue: int = EPI_STORE, force_splits: int = 0, packed_rows: Optional[int] = None) -> Optional[PartialSums]:
+                     epilogue: int = EPI_STORE, force_splits: int = 0, packed_rows: Optional[int] = None,
+                     alpha: float = 1.0) -> Optional[PartialSums]:
     """The same product, its sum left to the caller when it was cut along K: returns ``PartialSums`` ([splits][n][n_out]
-    float32 in a slab of the workspace; `out` is NOT written, and the bias not added) for the caller's next kernel
+    float32 in a slab of the workspace, `alpha` applied; `out` is NOT written, and the bias not added) for the caller's next kernel
     (``finish_*``) to sum, then ``release()``.  Returns None when the product was not cut: `out` is complete."""
-    r = _gemm_tc(x, w, out, bias, epilogue, ACT_NONE, force_splits, True, packed_rows)
+    r = _gemm_tc(x, w, out, bias, epilogue, ACT_NONE, force_splits, True, packed_rows, 0.0, alpha)
     return r if isinstance(r, PartialSums) else None
 
 
@@ -903,17 +905,18 @@ def mlstm(proj: torch.Tensor, cols, gates: torch.Tensor, state: torch.Tensor, co
     _count(3)
 
 
-def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, gate_col: int, w: torch.Tensor, y: torch.Tensor, H: int, V: int, eps: float,
+def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, gate_col: int, w: Optional[torch.Tensor], y: torch.Tensor, H: int, V: int, eps: float,
                    per_head_weight: bool = False, silu: bool = False) -> None:
     """y [n, H V] = o / rms(o per head) * w * act(gate[:, gate_col + h V + i]): o float32 [n, H V]; y in the activation dtype, gate
-    in y's dtype or float32; w float32, V values for all heads or (`per_head_weight`) H V; act the sigmoid, or SiLU with `silu`."""
+    in y's dtype or float32; w float32, V values for all heads or (`per_head_weight`) H V, or None (no weight); act the sigmoid, or SiLU with `silu`."""
     _dev(o, w, y)
     n = o.shape[0]
     assert o.dtype == torch.float32 and o.shape == (n, H * V) and y.shape == (n, H * V) and gate.stride(1) == 1
     assert gate.dtype in (y.dtype, torch.float32)
-    assert w.dtype == torch.float32 and w.numel() == (H * V if per_head_weight else V) and gate.shape[1] >= gate_col + H * V
+    assert w is None or (w.dtype == torch.float32 and w.numel() == (H * V if per_head_weight else V))
+    assert gate.shape[1] >= gate_col + H * V
     _check(lib().xr_head_norm_gate(o.data_ptr(), gate.data_ptr() + gate_col * gate.element_size(), dtype_code(gate.dtype), gate.stride(0),
-                                   w.data_ptr(), V if per_head_weight else 0, int(silu), y.data_ptr(), dtype_code(y.dtype), n, H, V,
+                                   _ptr(w), V if per_head_weight else 0, int(silu), y.data_ptr(), dtype_code(y.dtype), n, H, V,
                                    float(eps), _stream()), "head_norm_gate")
     _count()
 
@@ -953,13 +956,15 @@ def delta(proj: torch.Tensor, conv_w: torch.Tensor, gates: torch.Tensor, neg_a: 
 def route_topk(z: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, top: int, sigmoid_scores: bool = False,
                correction: Optional[torch.Tensor] = None) -> None:
     """ids[t], wts[t]: the `top` largest of z[t] (ties: lower index) and the softmax over them alone.  With `sigmoid_scores` the
-    scores are s = sigmoid(z): the `top` largest s + correction (float32 [E], optional) are chosen, and their weights are s as it is."""
-    _dev(z, ids, wts, correction)
+    scores are s = sigmoid(z): the `top` largest s + correction (float32 [E], optional) are chosen, and their weights are s as it is.
+    Rows of z may be strided (columns of a wider product)."""
+    _dev(ids, wts, correction)
+    assert z.is_cuda and z.stride(1) == 1
     assert correction is None or (sigmoid_scores and correction.dtype == torch.float32 and correction.numel() == z.shape[1])
     n, E = z.shape
     assert z.dtype == torch.float32 and ids.dtype == torch.int32 and wts.dtype == torch.float32
     assert ids.shape == (n, top) and wts.shape == (n, top)
-    _check(lib().xr_route_topk(z.data_ptr(), ids.data_ptr(), wts.data_ptr(), n, E, top, _ptr(correction), int(sigmoid_scores),
+    _check(lib().xr_route_topk(z.data_ptr(), z.stride(0), ids.data_ptr(), wts.data_ptr(), n, E, top, _ptr(correction), int(sigmoid_scores),
                                _stream()), "route_topk")
     _count()
 
@@ -1012,16 +1017,18 @@ def moe_gather(h: torch.Tensor, out: torch.Tensor, row_src, tile_group, top: int
 
 
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, row_src, tile_group, top: int,
-             gated: bool, act: int = ACT_NONE, limit: float = 0.0) -> None:
+             gated: bool, act: int = ACT_NONE, limit: float = 0.0, gather: Optional[bool] = None) -> None:
     """The experts' products over the planned rows (a plan with align = moe_tile_rows()), float32 FMA.  gated:
-    a = h [n, K], w [E, 2F, K], out [rows, F] = gate_act(h . w_gate, h . w_up); else a [rows, K], w [E, N, K], out [rows, N]."""
+    a = h [n, K], w [E, 2F, K], out [rows, F] = gate_act(h . w_gate, h . w_up); else a [rows, K], w [E, N, K], out [rows, N] = act(a . w),
+    or with `gather` a = h [n, K], every row taking its token's."""
     _dev(a, w, out)
+    gather = gated if gather is None else gather
     E, rows, K = w.shape
     N = rows // 2 if gated else rows
     assert a.shape[1] == K and out.shape[1] == N and out.shape[0] % moe_tile_rows() == 0
     _check(lib().xr_moe_gemm(a.data_ptr(), dtype_code(a.dtype), a.stride(0), w.data_ptr(), dtype_code(w.dtype), out.data_ptr(),
                              dtype_code(out.dtype), out.stride(0), row_src.data_ptr(), tile_group.data_ptr(),
-                             out.shape[0] // moe_tile_rows(), top, N, K, int(gated), int(act), float(limit), _stream()), "moe_gemm")
+                             out.shape[0] // moe_tile_rows(), top, N, K, int(gated), int(gather), int(act), float(limit), _stream()), "moe_gemm")
     _count()
 
 
@@ -1048,14 +1055,24 @@ def gemm_tc_grouped(x: torch.Tensor, w_packed: torch.Tensor, out: torch.Tensor, 
     _count()
 
 
-def moe_combine(d: torch.Tensor, z: torch.Tensor, wts: torch.Tensor, pair_row: torch.Tensor, top: int, h: Optional[torch.Tensor] = None) -> None:
-    """d[t] += sum_j wts[t, j] * z[pair_row[t * top + j]] (float32); a pair without a row (-1) adds wts[t, j] * h[t]."""
-    _dev(d, z, wts, pair_row)
+def moe_combine(d: torch.Tensor, z: torch.Tensor, wts: torch.Tensor, pair_row: torch.Tensor, top: int, h: Optional[torch.Tensor] = None,
+                shared: Optional[torch.Tensor] = None, splits: int = 1, gate: Optional[torch.Tensor] = None, scale: float = 1.0,
+                norm_w: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, eps: float = 0.0) -> None:
+    """d[t] += scale * (sum_j wts[t, j] * z[pair_row[t * top + j]] + sigmoid(gate[t]) * shared[t]) (float32); a pair without a row (-1)
+    adds wts[t, j] * h[t].  `shared` float32: [n, width], or [splits][n][width] partial sums; `gate` float32 [n] (may be strided; None:
+    the shared rows are added as they are).  With `norm_w` (float32 [width]) the new rows are normed in the same pass:
+    out[t] = d[t] / sqrt(mean(d[t]^2) + eps) * norm_w."""
+    _dev(d, z, wts, pair_row, shared, norm_w, out)
     n, width = d.shape
     assert d.dtype == torch.float32 and z.dtype == torch.float32 and z.shape[1] == width
     assert h is None or (h.is_cuda and h.shape == d.shape and h.stride(1) == 1)
+    assert shared is None or (shared.dtype == torch.float32 and splits >= 1 and shared.numel() >= splits * n * width)
+    assert gate is None or (shared is not None and gate.is_cuda and gate.dtype == torch.float32 and gate.shape == (n,))
+    assert (norm_w is None) == (out is None) and (out is None or (out.shape == d.shape and norm_w.dtype == torch.float32 and norm_w.numel() == width))
     _check(lib().xr_moe_combine(d.data_ptr(), z.data_ptr(), wts.data_ptr(), pair_row.data_ptr(), _ptr(h), 0 if h is None else dtype_code(h.dtype),
-                                0 if h is None else h.stride(0), n, width, top, _stream()), "moe_combine")
+                                0 if h is None else h.stride(0), _ptr(shared), int(splits), _ptr(gate), 0 if gate is None else gate.stride(0), float(scale),
+                                _ptr(norm_w), _ptr(out), 0 if out is None else dtype_code(out.dtype), float(eps), n, width, top, _stream()),
+           "moe_combine")
     _count()
 
 
@@ -1171,18 +1188,37 @@ def rglru(proj: torch.Tensor, conv_w, conv_b, wa_t, wi_t, wa, wi, ba, bi, lam, s
 
 
 def decay_attention(proj: torch.Tensor, cols, decay: torch.Tensor, state: torch.Tensor, seg_start, seg_len, seg_slot, o: torch.Tensor,
-                    n_seg: int, H: int, D: int, V: int) -> None:
-    """Linear attention with a constant decay per head: S <- decay_h S + k v^T, o = S^T q, with q, k, v = silu of proj's columns at
-    cols = (q, k, v); proj float32 [n, *] (a step of many tokens activates those columns in place), state float32 [slots, >= H D V],
-    o float32 [n, H V]."""
+                    n_seg: int, H: int, D: int, V: int, silu: bool = True, read_scale: float = 1.0) -> None:
+    """Linear attention with a constant decay per head: S <- decay_h S + k v^T, o = read_scale * S^T q, with q, k, v = proj's columns at
+    cols = (q, k, v), behind SiLU or (`silu` False) as they are; proj float32 [n, *] (a step of many tokens activates those columns in
+    place), state float32 [slots, >= H D V], o float32 [n, H V]."""
     _dev(decay, state, seg_start, seg_len, seg_slot, o)
     n = proj.shape[0]
     assert proj.dtype == torch.float32 and proj.stride(1) == 1 and o.shape == (n, H * V) and o.dtype == torch.float32
     assert decay.dtype == torch.float32 and decay.numel() == H and state.dtype == torch.float32 and state.shape[1] >= H * D * V
     _check(lib().xr_decay_attention(proj.data_ptr(), proj.stride(0), cols[0], cols[1], cols[2], decay.data_ptr(), state.data_ptr(),
                                     state.stride(0), seg_start.data_ptr(), seg_len.data_ptr(), seg_slot.data_ptr(), o.data_ptr(), n, n_seg, H, D, V,
-                                    _stream()), "decay_attention")
-    _count(2 if n > 16 else 1)
+                                    int(silu), float(read_scale), _stream()), "decay_attention")
+    _count(2 if silu and n > 16 else 1)
+
+
+def key_decay_attention(proj: torch.Tensor, cols, inner: int, w_t: torch.Tensor, bias: torch.Tensor, tau: float, decays: torch.Tensor,
+                        state: torch.Tensor, seg_start, seg_len, seg_slot, o: torch.Tensor, n_seg: int, H: int, D: int, V: int,
+                        read_scale: float = 1.0) -> None:
+    """Linear attention with a decay per key channel and token: S <- diag(a) S + k v^T, o = read_scale * S^T q, a = sigmoid(z)^(1/tau),
+    z = w_t^T proj[:, cols[3] : cols[3] + inner] + bias.  proj float32 [n, *]: q, k, v and the decays' inner values at
+    cols = (q, k, v, inner); w_t float32 [inner, H D], bias float32 [H D]; decays float32 [n, H D] scratch; state float32
+    [slots, >= H D V], o float32 [n, H V]."""
+    _dev(w_t, bias, decays, state, seg_start, seg_len, seg_slot, o)
+    n = proj.shape[0]
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and o.shape == (n, H * V) and o.dtype == torch.float32
+    assert w_t.dtype == torch.float32 and w_t.shape == (inner, H * D) and bias.dtype == torch.float32 and bias.numel() == H * D
+    assert decays.dtype == torch.float32 and decays.numel() >= n * H * D and proj.shape[1] >= cols[3] + inner
+    assert state.dtype == torch.float32 and state.shape[1] >= H * D * V
+    _check(lib().xr_key_decay_attention(proj.data_ptr(), proj.stride(0), cols[0], cols[1], cols[2], cols[3], w_t.data_ptr(), bias.data_ptr(), int(inner),
+                                        float(tau), decays.data_ptr(), state.data_ptr(), state.stride(0), seg_start.data_ptr(), seg_len.data_ptr(),
+                                        seg_slot.data_ptr(), o.data_ptr(), n, n_seg, H, D, V, float(read_scale), _stream()), "key_decay_attention")
+    _count(2)
 
 
 def ssd_state_floats(H: int, G: int, N: int, V: int, taps: int) -> int:

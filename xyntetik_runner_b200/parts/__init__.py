@@ -3,7 +3,7 @@ from .base import (Block, FeedForward, KVNeed, Mixer, Norm, Part, PositionEncodi
                    register_block, register_feed_forward, register_mixer, register_norm, register_position)
 from .attention import GQAAttention
 from .block import OutputNormBlock, ParallelBlock, PreNormBlock
-from .decay_attention import DecayLinearAttention
+from .decay_attention import DecayLinearAttention, KeyDecayLinearAttention
 from .delta import GatedDelta
 from .embedding import Embedding, Head, PairEmbedding
 from .feed_forward import GatedFeedForward, MLP, SwiGLU

@@ -28,7 +28,9 @@ differs from the other order when the position encoding scales its cosines and s
 value of position j is turned by j over all its Vd elements (pair m by j base^(-2m/Vd)) before it is cached, and every head's sum
 at position i is turned back by -i, so that what a query reads of a value depends on their distance.  `softcap` c: every scaled
 score s becomes c tanh(s / c).  `sink=0.0` (a number instead of a tensor's name): a sink of that logit for every head, which adds
-exp(sink) to every softmax's denominator.  `out_scale` multiplies the heads' outputs before the output product.
+exp(sink) to every softmax's denominator.  `out_scale` multiplies what the mixer adds to the stream: a factor on the output
+product's float32 sums (with rotated values: on the heads' sums as they are turned back).  `exact_angles`: the general path even where
+nothing else asks for it, for its rotation angles (float64 products of position and frequency).
 
 `keep_first` n (with a window): a request's first n keys stay visible behind the window, in their own positions; the pages that
 hold them stay held.  `distance_bias=(name, far)`: a learned table [rows, H] by distance joins the scaled scores, row
@@ -70,7 +72,7 @@ class GQAAttention(Mixer):
                  q_temp: Optional[tuple] = None, sink=None, gate: Optional[str] = None, g: str = "g",
                  norm_after_rotation: bool = False, value_rotation: Optional[tuple] = None, softcap: Optional[float] = None,
                  out_scale: float = 1.0, keep_first: int = 0, distance_bias: Optional[tuple] = None,
-                 value_share: Optional[str] = None, v_mix: str = "vmix"):
+                 value_share: Optional[str] = None, v_mix: str = "vmix", exact_angles: bool = False):
         if heads % kv_heads:
             raise ValueError("heads must be a multiple of kv_heads")
         if qk_norm not in (False, True, "unit"):
@@ -93,9 +95,9 @@ class GQAAttention(Mixer):
             raise ValueError(f"{prefix}: keep_first {keep_first}")
         self.D = head_dim                                      # query/key elements per head
         self.Vd = head_dim if value_dim is None else value_dim  # value elements per head
-        # the general path: a norm per head, or values of another size than keys
+        # the general path: a norm per head, values of another size than keys, or angles that must be float64 products
         self.general = bool(qk_norm) or self.Vd != self.D or q_temp is not None or gate is not None or \
-            value_rotation is not None or value_share is not None
+            value_rotation is not None or value_share is not None or bool(exact_angles)
         # head size of the cache and of the attention kernels
         hd = -(-max(self.D, self.Vd) // 16) * 16 if self.general else head_dim
         if not (1 <= hd <= 256):
@@ -113,7 +115,9 @@ class GQAAttention(Mixer):
         self.sink_value = float(sink) if sink is not None and not isinstance(sink, str) else None
         self.norm_after, self.value_rotation = bool(norm_after_rotation), value_rotation
         self.softcap = float(softcap) if softcap else 0.0
+        # the factor on the mixer's output rides in the output product (where the sums are turned back first, in that kernel)
         self.out_scale = float(out_scale)
+        self.alpha = 1.0 if value_rotation is not None else self.out_scale
         self.keep_first = int(keep_first) if window is not None else 0
         self.bias_name, self.bias_far = (None, 0.0) if distance_bias is None else (prefix + distance_bias[0], float(distance_bias[1]))
         if distance_bias is not None and not self.scale > 0:
@@ -172,6 +176,8 @@ class GQAAttention(Mixer):
                 bias = torch.cat([bias, torch.zeros(self.gate_cols, dtype=torch.float32, device=bias.device)])
         if self.out_bias:
             obias = tensors[o + self.bias_suffix]
+            if self.alpha != 1.0:
+                obias = obias.to(torch.float32) * self.alpha
         if self.sink_name is not None:
             self.sink = tensors[self.sink_name].to(torch.float32).contiguous()
         elif self.sink_value is not None:
@@ -307,15 +313,7 @@ class GQAAttention(Mixer):
             # the sums are turned back by their own position (and scaled in the same pass)
             kernels.rotate_heads(o, 0, self.H, self.hd, self.Vd, self.Vd, self.value_rotation[1] == "adjacent", self.vfreq64, ctx.positions,
                                  sign=-1.0, scale=self.out_scale)
-        elif self.out_scale != 1.0:
-            kernels.rotate_heads(o, 0, self.H, self.hd, 0, self.hd, False, self.freq64 if self.freq64 is not None else self._no_freq(o),
-                                 ctx.positions, scale=self.out_scale)
-        ctx.set_pending(x, self.out.forward(o, x, accumulate=True, defer=True))
-
-    def _no_freq(self, like):
-        if getattr(self, "_empty_freq", None) is None:
-            self._empty_freq = torch.zeros(1, dtype=torch.float64, device=like.device)
-        return self._empty_freq
+        ctx.set_pending(x, self.out.forward(o, x, accumulate=True, defer=True, alpha=self.alpha))
 
 
 register_mixer("gqa_attention", GQAAttention)

@@ -1,19 +1,23 @@
 """Pre-norm block: x -> norm -> mixer -> +x -> norm -> feed-forward -> +x
 (src/model.c:6206-6208, 6350-6352, 6366-6368, 6421-6423).  The two additions happen in float32
-inside the last product of the mixer and of the feed-forward."""
+inside the last product of the mixer and of the feed-forward (a factor on what a sublayer adds is the sublayer's `out_scale`)."""
 from __future__ import annotations
 
 import torch
 
+from ..weights.loader import TensorSpec
 from .base import Block, FeedForward, Mixer, Norm, register_block
+from .linear_tc import Pending
 from .norm import RMSNorm, ScalarRMSNorm
 
 
 class PreNormBlock(Block):
-    def __init__(self, mixer_norm: Norm, mixer: Mixer, ff_norm: Norm = None, feed_forward: FeedForward = None):
-        """`feed_forward` None: a layer of the mixer alone (no second norm either)."""
+    def __init__(self, mixer_norm: Norm, mixer: Mixer, ff_norm: Norm = None, feed_forward: FeedForward = None, spare_norm: str = None):
+        """`feed_forward` None: a layer of the mixer alone (no second norm either; `spare_norm` names the weight of one that a checkpoint
+        may carry all the same and nothing reads)."""
         if (ff_norm is None) != (feed_forward is None):
             raise ValueError("a feed-forward and its norm come together")
+        self.spare_norm = spare_norm
         self.mixer_norm, self.mixer, self.ff_norm, self.feed_forward = mixer_norm, mixer, ff_norm, feed_forward
 
     def parts(self):
@@ -27,6 +31,8 @@ class PreNormBlock(Block):
         out = {}
         for p in self.parts():
             out.update(p.tensors())
+        if self.spare_norm is not None:
+            out[self.spare_norm] = TensorSpec((self.mixer_norm.width,), kind="vector", init="ones", optional=True)
         return out
 
     def bind(self, tensors, rt):
@@ -176,6 +182,9 @@ class OutputNormBlock(Block):
         """x += norm(d); partial sums that the sublayer's last products left on d are taken in the same pass."""
         from .. import kernels
         pend = ctx.take_pending(d)
+        if pend is not None and not isinstance(pend, Pending):
+            pend.finish()
+            pend = None
         if pend is None:
             kernels.norm_add(d, x, norm.gain, norm.eps, cast=cast, clear=True)
             return

@@ -2,7 +2,7 @@
 
 Embedding: x[t] = E[id_t], ids outside the table read row 0, no scale (src/model.c:6148-6162).
 Head: logits = W_out . norm(x) at the wanted rows; when the model ties its head to the embedding
-the same tensor serves both (src/model.c:2353-2354).
+the same tensor serves both (src/model.c:2353-2354).  The logits may carry a factor and a cap.
 """
 from __future__ import annotations
 
@@ -71,11 +71,11 @@ class Head(Part):
     graph_safe = True
     """`tied_to` set: no tensor of its own, multiplies by the embedding table."""
 
-    def __init__(self, vocab: int, width: int, name: str = None, tied_to: Embedding = None, softcap: float = None):
-        """`softcap` c: the logits become c tanh(logits / c) (None or 0: as they are)."""
+    def __init__(self, vocab: int, width: int, name: str = None, tied_to: Embedding = None, softcap: float = None, scale: float = 1.0):
+        """`scale` multiplies the logits; `softcap` c: they then become c tanh(logits / c) (None or 0: as they are)."""
         assert (name is None) != (tied_to is None)
         self.vocab, self.width, self.name, self.tied_to = vocab, width, name, tied_to
-        self.softcap = float(softcap) if softcap else None
+        self.softcap, self.scale = float(softcap) if softcap else None, float(scale)
         self.linear = None
 
     def tensors(self):
@@ -90,6 +90,6 @@ class Head(Part):
         return self.linear.nbytes()
 
     def forward(self, ctx, h: torch.Tensor, logits: torch.Tensor) -> None:
-        self.linear.forward(h, logits)
+        self.linear.forward(h, logits, alpha=self.scale)
         if self.softcap is not None:
             kernels.softcap(logits, self.softcap)

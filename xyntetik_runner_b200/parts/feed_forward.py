@@ -86,10 +86,18 @@ class MLP(FeedForward):
     def weight_bytes(self):
         return self.up.nbytes() + self.down.nbytes()
 
-    def forward(self, ctx, h, x):
+    def _inner(self, ctx, h):
         act = ctx.buf("ffn_act", (h.shape[0], self.inner), ctx.act_dtype)
         self.up.forward(h, act, act=self.act)          # the activation rides in the product's epilogue
-        ctx.set_pending(x, self.down.forward(act, x, accumulate=True, defer=True))
+        return act
+
+    def forward(self, ctx, h, x):
+        ctx.set_pending(x, self.down.forward(self._inner(ctx, h), x, accumulate=True, defer=True))
+
+    def product(self, ctx, h, rows):
+        """The feed-forward's output into `rows` (float32) instead of the stream; a product cut along K returns its partial sums
+        (``linear_tc.Pending``) and leaves `rows` as they are."""
+        return self.down.forward(self._inner(ctx, h), rows, defer=True)
 
 
 register_feed_forward("swiglu", SwiGLU)

@@ -1,6 +1,6 @@
 """A weight matrix and the choice of kernel that multiplies by it.
 
-``out[t][r] (+)= sum_k x[t][k] W[r][k] (+ bias[r])``.  W keeps its stored dtype.  bfloat16 activations times
+``out[t][r] (+)= alpha sum_k x[t][k] W[r][k] (+ bias[r])``.  W keeps its stored dtype.  bfloat16 activations times
 a bfloat16 matrix go to the tensor-core kernel (tcgen05); for that the matrix is re-laid tile by tile when the
 part binds it (``prepare``), so that every tile the kernel streams is one contiguous read.  Everything else
 -- the true 32-bit path above all -- goes to the float32 FMA kernel on the matrix as stored.  Which kernel
@@ -43,19 +43,19 @@ class Linear:
         return self._nbytes
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, accumulate: bool = False, defer: bool = False,
-                act: int = kernels.ACT_NONE):
-        """out (+)= act(x W^T + bias) (an activation only without `accumulate`).  With `defer`, a product that was
+                act: int = kernels.ACT_NONE, alpha: float = 1.0):
+        """out (+)= act(alpha x W^T + bias) (an activation only without `accumulate`; `alpha` multiplies the float32 sums).  With `defer`, a product that was
         split along K leaves its partial sums in a slab of the workspace and returns ``Pending``; the caller's next
         kernel sums them (and adds the bias) and releases the slab.  Otherwise returns None and `out` is complete."""
         assert self.halves == 1, "a matrix of two halves is multiplied by forward_gated"
         assert act == kernels.ACT_NONE or not (accumulate or defer)
         if self.packed is not None or linear_tc.usable(self, x, out, accumulate):
             counters["tcgen05"] += 1
-            pending = linear_tc.run(self, x, out, accumulate, defer, act)
+            pending = linear_tc.run(self, x, out, accumulate, defer, act, alpha)
             if pending is not None:
                 counters["deferred"] += 1
             return pending
-        kernels.gemm_simt(x, self.weight, out, self.bias, accumulate)
+        kernels.gemm_simt(x, self.weight, out, self.bias, accumulate, alpha)
         if act != kernels.ACT_NONE:
             kernels.act_mul(out, out, act, gated=False)
         counters["simt"] += 1

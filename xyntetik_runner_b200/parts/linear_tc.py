@@ -27,6 +27,11 @@ class Pending:
         kernels.finish_plain(self.partial, self.splits, self.bias, self.out, self.accumulate)
         self.release()
 
+    def finish_norm(self, x, w, out, eps, w2=None, out2=None) -> None:
+        """The sum added into x and the norm of the new rows into `out` (and with `w2` into `out2`), in one pass."""
+        kernels.finish_add_rmsnorm(self.partial, self.splits, self.bias, x, w, out, eps, w2, out2)
+        self.release()
+
     def join(self, later: "Pending") -> Optional["Pending"]:
         """One pending sum for this product's and a later one's, when both add into the same rows, their slabs lie one right
         behind the other and at most one has a bias: the partial sums then read as one array [splits + later.splits][n][width],
@@ -59,14 +64,14 @@ def usable(lin, x, out, accumulate) -> bool:
     return ENABLED and lin.weight is not None and kernels.gemm_tc_supported(x, lin.weight, out)
 
 
-def run(lin, x, out, accumulate, defer=False, act=kernels.ACT_NONE):
+def run(lin, x, out, accumulate, defer=False, act=kernels.ACT_NONE, alpha=1.0):
     epi = kernels.EPI_ADD if accumulate else kernels.EPI_STORE
     w, packed_rows = (lin.packed, lin.n_out) if lin.packed is not None else (lin.weight, None)
     if defer:
         assert act == kernels.ACT_NONE
-        sums = kernels.gemm_tc_deferred(x, w, out, lin.bias, epi, packed_rows=packed_rows)
+        sums = kernels.gemm_tc_deferred(x, w, out, lin.bias, epi, packed_rows=packed_rows, alpha=alpha)
         if sums is None:
             return None
         return Pending(sums, lin.bias, out, accumulate)
-    kernels.gemm_tc(x, w, out, lin.bias, epi, packed_rows=packed_rows, act=act)
+    kernels.gemm_tc(x, w, out, lin.bias, epi, packed_rows=packed_rows, act=act, alpha=alpha)
     return None

@@ -36,9 +36,8 @@ class RMSNorm(Norm):
             w2 = second.weight
         pend = ctx.take_pending(x)
         if pend is not None and rows is None:
-            # the product before this norm left partial sums: sum, add into x and normalise in one pass
-            kernels.finish_add_rmsnorm(pend.partial, pend.splits, pend.bias, x, self.weight, out, self.eps, w2, out2)
-            pend.release()
+            # the part before this norm left its last sum: sum, add into x and normalise in one pass
+            pend.finish_norm(x, self.weight, out, self.eps, w2, out2)
             return
         if pend is not None:
             pend.finish()

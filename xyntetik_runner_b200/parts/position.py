@@ -22,18 +22,18 @@ import torch
 from .base import PositionEncoding, Rotary, register_position
 
 
-def llama3_divisors(inv_freq: np.ndarray, factor: float, low: float, high: float, orig: int) -> np.ndarray:
-    out = np.ones_like(inv_freq, dtype=np.float32)
+def llama3_divisors(inv_freq: np.ndarray, factor: float, low: float, high: float, orig: float, dtype=np.float32) -> np.ndarray:
+    out = np.ones_like(inv_freq, dtype=dtype)
     for j, f in enumerate(inv_freq.tolist()):
         lam = 2.0 * math.pi / f
         if lam < orig / high:
             d = 1.0
-        elif lam > orig / low:
+        elif low > 0 and lam > orig / low or high <= low:
             d = factor
         else:
             s = (orig / lam - low) / (high - low)
             d = f / ((1.0 - s) * f / factor + s * f)
-        out[j] = np.float32(d)
+        out[j] = d
     return out
 
 
@@ -91,13 +91,17 @@ class Rope(PositionEncoding):
             inv = (inv / div).astype(np.float32)
         self.inv_freq_host = inv
         self.inv_freq = None
-        # the same frequencies in float64, for kernels that take the angle in float64 (unscaled or linearly scaled frequencies only)
+        # the same frequencies in float64, for kernels that take the angle in float64
         self.inv_freq64_host = None
         linear = scaling is not None and getattr(scaling, "rope_type", "llama3") == "linear"
-        if (scaling is None or linear) and half:
+        if half:
             self.inv_freq64_host = np.power(float(theta), -2.0 * np.arange(half, dtype=np.float64) / float(self.rotary_dim))
             if linear:
                 self.inv_freq64_host = self.inv_freq64_host / float(scaling.factor)
+            elif scaling is not None:
+                self.inv_freq64_host = self.inv_freq64_host / llama3_divisors(
+                    self.inv_freq64_host, scaling.factor, scaling.low_freq_factor, scaling.high_freq_factor,
+                    scaling.original_max_position_embeddings, np.float64)
 
     def prepare(self, rt):
         self.inv_freq = torch.from_numpy(self.inv_freq_host.copy()).to(rt.device)

@@ -32,6 +32,7 @@ class TensorSpec:
     init: str = "normal"          # random mode: "normal" | "ones" | "ones_jitter" | "zeros" | "zeros_jitter"
     optional: bool = False        # a source may lack it (the model then never reads it); random sources leave it out
     any_rows: bool = False        # the source says how many rows there are; shape[0] is what random sources make
+    any_cols: bool = False        # the same for the last axis
 
 
 class WeightsError(ValueError):
@@ -165,8 +166,9 @@ def load_tensors(expected: Mapping[str, TensorSpec], source: TensorSource,
             continue
         dt, shape = have[n]
         same = tuple(shape) == tuple(spec.shape)
-        if spec.any_rows:
-            same = len(shape) == len(spec.shape) and shape[0] >= 1 and tuple(shape[1:]) == tuple(spec.shape[1:])
+        if spec.any_rows or spec.any_cols:
+            free = ([0] if spec.any_rows else []) + ([len(spec.shape) - 1] if spec.any_cols else [])
+            same = len(shape) == len(spec.shape) and all(shape[a] >= 1 if a in free else shape[a] == spec.shape[a] for a in range(len(shape)))
         if not same:
             wrong.append((n, tuple(shape), tuple(spec.shape)))
         if spec.kind == "table":
