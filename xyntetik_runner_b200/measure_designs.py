@@ -1,5 +1,5 @@
-"""Prefill and decode throughput of a Turudra, a Besolix, a Pitolix, a Buzarax or a Semesun model beside a dense Llama of equal size (Semesun:
-also beside a Buzarax model, whose recurrences and experts are the nearest to its own), with the time of every kernel family inside the
+"""Prefill and decode throughput of a Turudra, a Besolix, a Pitolix, a Buzarax, a Semesun or a Lilalorn model beside a dense Llama of equal
+size (Semesun and Lilalorn: also beside a Buzarax model, whose recurrences and experts are the nearest to their own), with the time of every kernel family inside the
 steps (``bench.py --designs``).
 
 Sizes resemble real layers; weights are random.  Both models run through the same engine: one prompt of `tokens` tokens
@@ -22,6 +22,7 @@ import torch
 from . import kernels, measure
 from .config.besolix import BesolixConfig
 from .config.buzarax import BuzaraxConfig
+from .config.lilalorn import LilalornConfig
 from .config.llama import LlamaConfig
 from .config.pitolix import PitolixConfig
 from .config.semesun import SemesunConfig
@@ -181,6 +182,37 @@ def llama_like_semesun(size: str, positions: int) -> LlamaConfig:
                                   "max_position_embeddings": positions, "torch_dtype": "bfloat16"})
 
 
+LILALORN_SIZES = {
+    # name: (width, softmax side (heads, kv heads, head size, rotated elements), retention (heads, key size, value size), gated linear
+    # attention (heads, key size, value size), experts, chosen, expert feed-forward, shared feed-forward, vocab); six layers: the
+    # parallel mixer and gated linear attention in turn
+    "lilalorn-w1024": (1024, (8, 2, 128, 128), (4, 128, 128), (4, 128, 256), 16, 2, 1408, 1408, 32000),
+    "lilalorn-w2048": (2048, (16, 4, 128, 128), (8, 128, 128), (8, 128, 256), 16, 2, 2816, 2816, 32000),
+}
+
+
+def lilalorn_config(size: str) -> LilalornConfig:
+    W, (H, K, D, rot), (rh, rd, rv), (gh, gd, gv), E, top, eff, sff, vocab = LILALORN_SIZES[size]
+    moe = {"kind": "moe", "router": {"experts": E, "top": top}, "expert": {"ff": eff}, "shared": {"ff": sff}}
+    par = {"type": "parallel", "mlp": moe, "mixer": {
+        "left": {"heads": H, "kv_heads": K, "dim": D, "vdim": D, "scale": D ** -0.5,
+                 "rot": {"base": 200000.0, "dims": rot, "scaling": {"factor": 16.0, "low": 1.0, "high": 8.0, "original": 4096}}},
+        "right": {"heads": rh, "dim": rd, "vdim": rv, "decay": [1.0 - 2.0 ** -(3 + 5.0 * h / max(rh - 1, 1)) for h in range(rh)]},
+        "left_scale": 0.7, "right_scale": 0.9}}
+    gla = {"type": "gla", "mlp": moe, "mixer": {"heads": gh, "dim": gd, "vdim": gv, "tau": 12.0}}
+    return LilalornConfig.from_dict({"architecture": "Lilalorn", "vocab": vocab, "width": W, "norm": {"eps": 1e-5}, "residual_mult": 0.7,
+                                     "logit_scale": 0.8, "layers": [par, gla, par, gla, par, gla]})
+
+
+def llama_like_lilalorn(size: str, positions: int) -> LlamaConfig:
+    """A dense decoder of the same width, number of layers and attention heads, its feed-forward as wide as what a token uses."""
+    W, (H, K, D, rot), _, _, E, top, eff, sff, vocab = LILALORN_SIZES[size]
+    return LlamaConfig.from_dict({"architectures": ["LlamaForCausalLM"], "hidden_size": W, "num_hidden_layers": 6,
+                                  "num_attention_heads": H, "num_key_value_heads": K, "head_dim": D,
+                                  "intermediate_size": 2 * (top * eff + sff) // 3, "vocab_size": vocab, "rms_norm_eps": 1e-5, "rope_theta": 10000.0,
+                                  "max_position_embeddings": positions, "torch_dtype": "bfloat16"})
+
+
 FAMILIES = {
     "gemm_tc": "products (tcgen05)", "gemm_tc_deferred": "products (tcgen05)", "gemm_simt": "products (FMA)",
     "finish_plain": "products (tcgen05)", "finish_add_rmsnorm": "norms", "rmsnorm": "norms", "finish_rope_store": "rotation + cache store",
@@ -193,7 +225,7 @@ FAMILIES = {
     "delta": "delta recurrence", "head_norm_gate": "delta recurrence", "qk_norm_rope_store": "rotation + cache store",
     "rmsnorm_act": "norms", "ssd": "state-space recurrence", "silu_gate_norm": "gated norm of the recurrence", "route_groups": "routing",
     "sigmoid_gate": "output gates", "stream_step": "stream kernels",
-    "rglru": "gated linear recurrence", "decay_attention": "decay attention recurrence", "norm_add": "norms", "depth_average": "stream kernels",
+    "rglru": "gated linear recurrence", "decay_attention": "decay attention recurrence", "key_decay_attention": "key-decay attention recurrence", "norm_add": "norms", "depth_average": "stream kernels",
     "cast_rows": "stream kernels", "row_norm_gate": "decay attention recurrence", "embed_pair": "stream kernels", "last_token": "stream kernels", "rotate_heads": "rotation + cache store",
     "scaled_add": "stream kernels", "concat_cast": "stream kernels", "softcap": "stream kernels", "embed": "stream kernels", "act_mul": "stream kernels",
 }
@@ -439,6 +471,51 @@ def _semesun_work(cfg, tokens, keys_per_token, decode):
             "experts' sum": (0.0, by_c)}
 
 
+def _lilalorn_work(cfg, tokens, keys_per_token, decode):
+    """(FLOPs, bytes) per kernel family in one step of `tokens` tokens, counted like ``_buzarax_work``."""
+    W = cfg.width
+    fl_a = by_a = fl_p = by_p = by_n = by_r = fl_d = by_d = fl_k = by_k = by_h = fl_e = by_e = by_c = 0.0
+    once = tokens if decode else 1
+    for lay in cfg.layers:
+        m = lay.mixer
+        if m.kind == "parallel":
+            l, r = m.left, m.right
+            hd = max(l.dim, l.vdim)
+            cols = (l.heads + l.kv_heads) * l.dim + l.kv_heads * l.vdim
+            rcols = 2 * r.heads * r.dim + 2 * r.heads * r.vdim
+            per = W * (cols + rcols) + (l.heads * l.vdim + r.heads * r.vdim) * W
+            fl_a += 2.0 * tokens * l.heads * keys_per_token * (l.dim + l.vdim)
+            by_a += once * keys_per_token * 2 * l.kv_heads * hd * 2
+            by_r += tokens * 2.0 * (cols + (l.heads + 2 * l.kv_heads) * hd)
+            # per token and state element: decay and update, read-out; the state once per request and step, the rows in float32
+            fl_d += 4.0 * tokens * r.heads * r.dim * r.vdim
+            by_d += once * 2 * r.heads * r.dim * r.vdim * 4 + tokens * (2 * r.heads * r.dim + 2 * r.heads * r.vdim) * 4
+            by_h += tokens * r.heads * r.vdim * (4 + 4 + 2.0)
+        else:
+            HD, HV = m.heads * m.dim, m.heads * m.vdim
+            per = W * (2 * HD + 2 * HV + 16) + HV * W
+            fl_k += tokens * (4.0 * HD * m.vdim + 2.0 * 16 * HD)
+            # the decays are written once and read by the walk
+            by_k += once * 2 * HD * m.vdim * 4 + tokens * (4 * HD + 2 * HV) * 4
+            by_h += tokens * HV * (4 + 4 + 2.0)
+        f = lay.mlp
+        if f is not None:
+            fl_e += 2.0 * tokens * f.top * 2 * f.ff * W
+            by_e += min(f.experts, tokens * f.top) * 2 * f.ff * W * 2
+            per += (f.experts + 1) * W + 2 * (f.shared_ff or 0) * W
+            # the chosen rows, the shared expert's, the stream in and out, and the norm's row
+            by_c += tokens * W * (4.0 * (f.top + 1 + 2) + 2)
+        fl_p += 2.0 * tokens * per
+        by_p += 2.0 * per
+        by_n += tokens * W * (4 + 2)
+    fl_p += 2.0 * cfg.vocab * W * (tokens if decode else 1)
+    by_p += 2.0 * cfg.vocab * W
+    by_n += tokens * W * (4 + 2)
+    return {"attention": (fl_a, by_a), "products (tcgen05)": (fl_p, by_p), "norms": (0.0, by_n), "rotation + cache store": (0.0, by_r),
+            "decay attention recurrence": (fl_d, by_d), "key-decay attention recurrence": (fl_k, by_k), "delta recurrence": (0.0, by_h),
+            "grouped products (experts, per-head)": (fl_e, by_e), "experts' sum": (0.0, by_c)}
+
+
 def _measure(eng, cfg, work_fn, tokens: int, batch: int, context: int, steps: int, warmup: int, pk, phase: str = "both") -> dict:
     vocab = eng.plan.vocab_size
     gen = torch.Generator().manual_seed(0)
@@ -529,6 +606,10 @@ def compare(size: str, tokens: int = 2048, batch: int = 8, context: int = 2048, 
         near = size.replace("semesun", "buzarax")
         arms = (("semesun", semesun_config(size), _semesun_work), ("buzarax", buzarax_config(near), _buzarax_work),
                 ("llama", llama_like_semesun(size, context + tokens), _llama_window_work))
+    elif size in LILALORN_SIZES:
+        near = size.replace("lilalorn", "buzarax")
+        arms = (("lilalorn", lilalorn_config(size), _lilalorn_work), ("buzarax", buzarax_config(near), _buzarax_work),
+                ("llama", llama_like_lilalorn(size, context + tokens), _llama_work))
     elif size in BUZARAX_SIZES:
         arms = (("buzarax", buzarax_config(size), _buzarax_work), ("llama", llama_like_buzarax(size, context + tokens), _llama_work))
     elif size in PITOLIX_SIZES:
@@ -540,7 +621,7 @@ def compare(size: str, tokens: int = 2048, batch: int = 8, context: int = 2048, 
         arms = (("turudra", tcfg, _work), ("llama", llama_config(size, len(tcfg.layer_runs()), context + tokens), _llama_work))
     for name, cfg, work in arms:
         # (`models` names arms to run; "turudra" also stands for the new design's arm of a Besolix size: the default runs both arms)
-        if name not in models and not (name in ("besolix", "pitolix", "buzarax", "semesun") and "turudra" in models):
+        if name not in models and not (name in ("besolix", "pitolix", "buzarax", "semesun", "lilalorn") and "turudra" in models):
             continue
         t0 = time.perf_counter()
         eng = random_engine(cfg, 5, ep())
