@@ -309,14 +309,13 @@ XR_EXPORT int xr_rglru(float* proj, long long ldp, int y_col, int x_col, const f
 // and adds them, times q, into VC sums.  The sums of 32 / VC tokens are added over the lanes together: 32 numbers a lane, halved
 // five times by an exchange with the lane 16, 8, 4, 2, 1 away, after which every lane holds one (token, column) sum and stores
 // it: 31 shuffles for 32 / VC tokens, and one chain of five exchanges instead of one per token.
-// The tokens' q, k and v come in chunks of CH tokens through shared memory, two buffers: the next chunk's values are fetched into
-// registers before this chunk is walked and stored behind it (16 bytes a load where sizes and addresses allow: VEC).  A step of
-// many tokens applies silu to the rows beforehand, in
-// place (k_silu_cols); a step of few applies it on the way into shared memory.
+// Two elements are updated at a time by packed float32 multiply-adds (f32x2).  The tokens' q, k and v come in chunks of CH tokens
+// through shared memory, two buffers: the next chunk's values are copied asynchronously while this chunk is walked (16 bytes a copy
+// where sizes and addresses allow: VEC).  A step of many tokens applies silu to the rows beforehand, in place (k_silu_cols); a step
+// of few applies it in shared memory.  A column's D state values lie together in memory ([H][V][D]), a lane's JD of them side by side.
 // KIND: DS_HEAD: a constant decay per head.  DS_KEY: a decay per key channel and token, rows [n][H D] of their own.
 // DS_SSD: the decay and the factor on the value come per token and head (coef), heads share key and query rows by `rep`, the
-// value times skip[h] joins the read-out, a column's state lies together in memory ([H][V][D] instead of [H][D][V]), and the
-// blocks of a portion leave the convolution's new tail behind the walk.
+// value times skip[h] joins the read-out, and the blocks of a portion leave the convolution's new tail behind the walk.
 #define DA_WARPS 8
 #define DS_HEAD 0
 #define DS_SSD 1
@@ -343,6 +342,35 @@ __global__ void k_silu_cols(float* __restrict__ rows, long long ld, int cols, si
     }
 }
 
+// Two floats in one 64-bit register, and the packed arithmetic on them (each half rounded as the scalar operation is).
+typedef unsigned long long F2;
+__device__ __forceinline__ F2 f2_pack(float lo, float hi) { F2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi)); return r; }
+__device__ __forceinline__ float2 f2_unpack(F2 v) { float2 r; asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v)); return r; }
+__device__ __forceinline__ F2 f2_mul(F2 a, F2 b) { F2 r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
+__device__ __forceinline__ F2 f2_fma(F2 a, F2 b, F2 c) { F2 r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
+
+template <int BYTES>
+__device__ __forceinline__ void rc_copy_async(float* dst, const float* src) {
+    const unsigned at = (unsigned)__cvta_generic_to_shared(dst);
+    if constexpr (BYTES == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(at), "l"(src) : "memory");
+    else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(at), "l"(src) : "memory");
+}
+__device__ __forceinline__ void rc_copy_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
+// A lane's values of one token (JD of them) as pairs (JD 1: the value twice)
+template <int JD>
+__device__ __forceinline__ void rc_lane_values(const float* row, int lane, F2* out) {
+    if constexpr (JD == 1) { const float x = row[lane]; out[0] = f2_pack(x, x); }
+    else if constexpr (JD == 2) out[0] = *reinterpret_cast<const F2*>(row + 2 * lane);
+    else {
+#pragma unroll
+        for (int j = 0; j < JD; j += 4) {
+            const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(row + lane * JD + j);
+            out[j / 2] = x.x; out[j / 2 + 1] = x.y;
+        }
+    }
+}
+
 template <int JD, int VC, int CH, bool VEC, int KIND>
 __global__ void __launch_bounds__(32 * DA_WARPS)
 k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col, int v_col, const float* __restrict__ decay,
@@ -351,9 +379,10 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
     xr_pdl_launch();
     constexpr bool SSD = KIND == DS_SSD, KEY = KIND == DS_KEY;
     // a token's row in shared memory: q [DP], k [DP] (zeros behind D), DS_KEY: its decays [DP], the block's v [COLS]
-    constexpr int COLS = VC * DA_WARPS, DP = 32 * JD, VA = (KEY ? 3 : 2) * DP, RW = VA + COLS, TB = 32 / VC;
-    constexpr int PER = (CH * RW + 32 * DA_WARPS - 1) / (32 * DA_WARPS);
-    static_assert(CH % TB == 0, "a chunk is whole batches of tokens");
+    constexpr int COLS = VC * DA_WARPS, DP = 32 * JD, VA = (KEY ? 3 : 2) * DP, RW = VA + COLS, TB = 32 / VC, THREADS = 32 * DA_WARPS;
+    // pairs: two neighbouring key channels of a lane (JD 1: two neighbouring value columns)
+    constexpr int NP = JD == 1 ? 1 : JD / 2, NC = JD == 1 ? VC / 2 : VC;
+    static_assert(CH % TB == 0 && VC % 2 == 0, "a chunk is whole batches of tokens");
     extern __shared__ __align__(16) float da_sm[];           // two chunks of CH rows
     __shared__ __align__(8) float da_coef[SSD ? 2 * CH * 2 : 2];       // SSD: a token's decay and dt
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -363,102 +392,105 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
     const float dec = KIND == DS_HEAD ? decay[h] : 0.f, skip = SSD ? ssd.skip[h] : 0.f;
     float* slot = state + (size_t)seg_slot[seg] * state_stride;
     float* st = slot + (size_t)h * D * V;
-    auto at = [&](int d, int c) -> size_t { return SSD ? (size_t)(v0 + c) * D + d : (size_t)d * V + v0 + c; };
-    xr_pdl_wait();
-    float s[VC][JD];
-    // (SSD: a lane's JD elements of a column lie together: one access where they fall on a border of their size)
-    const bool whole = SSD && JD > 1 && D % JD == 0 && ((uintptr_t)st % (JD >= 4 ? 16 : 8)) == 0;
-    if (whole) {
+    auto at = [&](int d, int c) -> size_t { return (size_t)(v0 + c) * D + d; };
+    // (a chunk's columns behind D, and those of value columns that do not exist, are never copied to)
+    if (D < DP || vb + COLS > V)
+        for (int e = threadIdx.x; e < 2 * CH * RW; e += THREADS) da_sm[e] = 0.f;
+    // ---- the copies of a chunk: 16 bytes each where sizes and addresses allow.  Where a thread's pieces lie is worked out once; a
+    // chunk further they lie CH rows further.
+    constexpr int UNIT = VEC ? 4 : 1, PIECES = CH * RW / UNIT, PER = (PIECES + THREADS - 1) / THREADS;
+    auto source = [&](int e, long long& step) -> const float* {
+        const int tok = e / RW, cc = e % RW;
+        const float* row = proj + (size_t)(start + tok) * ldp;
+        step = (long long)CH * ldp;
+        if (e >= CH * RW) return nullptr;
+        if (cc < DP) return cc < D ? row + q_col + g * D + cc : nullptr;
+        if (cc < 2 * DP) return cc - DP < D ? row + k_col + g * D + cc - DP : nullptr;
+        if (KEY && cc < VA) {
+            step = (long long)CH * H * D;
+            return cc - 2 * DP < D ? key.rows + ((size_t)(start + tok) * H + h) * D + cc - 2 * DP : nullptr;
+        }
+        return vb + cc - VA < V ? row + v_col + h * V + vb + cc - VA : nullptr;
+    };
+    const float* src[VEC ? PER : 1];
+    long long step[VEC ? PER : 1];
+    if constexpr (VEC) {
 #pragma unroll
-        for (int c = 0; c < VC; c++) {
-            const bool ok = lane * JD < D && v0 + c < V;
-            const float* p = st + at(lane * JD, ok ? c : 0);
-            if constexpr (JD % 4 == 0) {
+        for (int k = 0; k < PER; k++) src[k] = source(4 * (threadIdx.x + k * THREADS), step[k]);
+    }
+    auto load = [&](int chunk) {
+        float* dst = da_sm + (chunk & 1) * CH * RW;
+        if (SSD && threadIdx.x < 2 * CH) {
+            const int i = chunk * CH + threadIdx.x / 2;
+            if (i < len) rc_copy_async<4>(da_coef + (chunk & 1) * 2 * CH + threadIdx.x, ssd.coef + ((size_t)(start + i) * H + h) * 2 + (threadIdx.x & 1));
+        }
+        if constexpr (VEC) {
 #pragma unroll
-                for (int j = 0; j < JD; j += 4) {
-                    const float4 x = ok ? *reinterpret_cast<const float4*>(p + j) : make_float4(0.f, 0.f, 0.f, 0.f);
-                    s[c][j] = x.x; s[c][j + 1] = x.y; s[c][j + 2] = x.z; s[c][j + 3] = x.w;
+            for (int k = 0; k < PER; k++) {
+                const int e = 4 * (threadIdx.x + k * THREADS);
+                if (src[k] != nullptr) {
+                    if (chunk * CH + e / RW < len) rc_copy_async<16>(dst + e, src[k]);
+                    src[k] += step[k];
                 }
-            } else if constexpr (JD == 2) {
-                const float2 x = ok ? *reinterpret_cast<const float2*>(p) : make_float2(0.f, 0.f);
-                s[c][0] = x.x; s[c][1] = x.y;
             }
+        } else {
+            for (int e = threadIdx.x; e < CH * RW; e += THREADS) {
+                long long st1;
+                const float* p = chunk * CH + e / RW < len ? source(e, st1) : nullptr;
+                if (p != nullptr) rc_copy_async<4>(dst + e, p + chunk * st1);
+            }
+        }
+    };
+    // behind the wait a thread may read what it copied itself: the activation in place
+    auto arrive = [&](int chunk) {
+        rc_copy_wait();
+        if (!activated) {
+            float* dst = da_sm + (chunk & 1) * CH * RW;
+#pragma unroll 1
+            for (int k = 0; k < PER; k++) {
+                const int e = UNIT * (threadIdx.x + k * THREADS);
+                if (e < CH * RW && chunk * CH + e / RW < len)
+                    for (int i = 0; i < UNIT; i++) dst[e + i] = rc_silu(dst[e + i]);
+            }
+        }
+    };
+    xr_pdl_wait();
+    const int chunks = (len + CH - 1) / CH;
+    if (D < DP || vb + COLS > V) __syncthreads();            // (zeros stand before copies land beside them)
+    if (chunks > 0) load(0);
+    // ---- the state: a lane's JD elements of a column lie together: one access where they fall on a border of their size
+    F2 s[NC][NP];
+    const bool whole = JD > 1 && D % JD == 0 && ((uintptr_t)st % (JD >= 4 ? 16 : 8)) == 0;
+    if constexpr (JD == 1) {
+#pragma unroll
+        for (int c = 0; c < NC; c++) {
+            const bool a0 = lane < D && v0 + 2 * c < V, a1 = lane < D && v0 + 2 * c + 1 < V;
+            s[c][0] = f2_pack(a0 ? st[at(lane, 2 * c)] : 0.f, a1 ? st[at(lane, 2 * c + 1)] : 0.f);
         }
     } else {
 #pragma unroll
-        for (int j = 0; j < JD; j++) {
-            const int d = lane * JD + j;
+        for (int c = 0; c < VC; c++) {
+            const bool ok = v0 + c < V;
+            const float* p = st + at(lane * JD, ok ? c : 0);
 #pragma unroll
-            for (int c = 0; c < VC; c++) s[c][j] = (d < D && v0 + c < V) ? st[at(d, c)] : 0.f;
+            for (int j = 0; j < JD; j += 2) {
+                const int d = lane * JD + j;
+                if (whole && JD % 4 == 0) {
+                    if (j % 4 == 0) {
+                        const float4 x = ok && d < D ? *reinterpret_cast<const float4*>(p + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+                        s[c][j / 2] = f2_pack(x.x, x.y);
+                        if (j / 2 + 1 < NP) s[c][j / 2 + 1] = f2_pack(x.z, x.w);
+                    }
+                } else if (whole) {
+                    const float2 x = ok && d < D ? *reinterpret_cast<const float2*>(p + j) : make_float2(0.f, 0.f);
+                    s[c][j / 2] = f2_pack(x.x, x.y);
+                } else {
+                    s[c][j / 2] = f2_pack(ok && d < D ? p[j] : 0.f, ok && d + 1 < D ? p[j + 1] : 0.f);
+                }
+            }
         }
     }
-    float coef_stage = 0.f;
-    constexpr int PER4 = (CH * RW / 4 + 32 * DA_WARPS - 1) / (32 * DA_WARPS);
-    float stage[VEC ? 1 : PER];
-    float4 stage4[VEC ? PER4 : 1];
-    // (loads that stay where they are written: left alone, the compiler moves them down to their use behind the walk to save
-    // registers, and the chunk then waits for them one after the other)
-    auto load = [&](int chunk) {
-        if (SSD && threadIdx.x < 2 * CH) {
-            const int i = chunk * CH + threadIdx.x / 2;
-            coef_stage = i < len ? xr_ld_now(ssd.coef + ((size_t)(start + i) * H + h) * 2 + (threadIdx.x & 1)) : 0.f;
-        }
-        if constexpr (VEC) {
-#pragma unroll
-            for (int k = 0; k < PER4; k++) {
-                const int e = 4 * (threadIdx.x + k * 32 * DA_WARPS);
-                const int tok = e / RW, cc = e % RW, i = chunk * CH + tok;
-                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (tok < CH && i < len) {
-                    const float* row = proj + (size_t)(start + i) * ldp;
-                    if (cc < DP) { if (cc < D) v = xr_ld_now4(reinterpret_cast<const float4*>(row + q_col + g * D + cc)); }
-                    else if (cc < 2 * DP) { if (cc - DP < D) v = xr_ld_now4(reinterpret_cast<const float4*>(row + k_col + g * D + cc - DP)); }
-                    else if (KEY && cc < VA) { if (cc - 2 * DP < D) v = xr_ld_now4(reinterpret_cast<const float4*>(key.rows + ((size_t)(start + i) * H + h) * D + cc - 2 * DP)); }
-                    else if (vb + cc - VA < V) v = xr_ld_now4(reinterpret_cast<const float4*>(row + v_col + h * V + vb + cc - VA));
-                }
-                stage4[k] = v;
-            }
-#pragma unroll
-            for (int k = 0; k < PER4; k++) xr_ld_fence(stage4[k]);
-        } else {
-#pragma unroll
-            for (int k = 0; k < PER; k++) {
-                const int e = threadIdx.x + k * 32 * DA_WARPS;
-                const int tok = e / RW, cc = e % RW, i = chunk * CH + tok;
-                float v = 0.f;
-                if (tok < CH && i < len) {
-                    const float* row = proj + (size_t)(start + i) * ldp;
-                    if (cc < DP) { if (cc < D) v = xr_ld_now(row + q_col + g * D + cc); }
-                    else if (cc < 2 * DP) { if (cc - DP < D) v = xr_ld_now(row + k_col + g * D + cc - DP); }
-                    else if (KEY && cc < VA) { if (cc - 2 * DP < D) v = xr_ld_now(key.rows + ((size_t)(start + i) * H + h) * D + cc - 2 * DP); }
-                    else if (vb + cc - VA < V) v = xr_ld_now(row + v_col + h * V + vb + cc - VA);
-                }
-                stage[k] = v;
-            }
-#pragma unroll
-            for (int k = 0; k < PER; k++) xr_ld_fence(stage[k]);
-        }
-    };
-    auto store = [&](int buf) {
-        if (SSD && threadIdx.x < 2 * CH) da_coef[buf * 2 * CH + threadIdx.x] = coef_stage;
-        if constexpr (VEC) {
-#pragma unroll
-            for (int k = 0; k < PER4; k++) {
-                const int e = 4 * (threadIdx.x + k * 32 * DA_WARPS);
-                float4 v = stage4[k];
-                if (!activated) { v.x = rc_silu(v.x); v.y = rc_silu(v.y); v.z = rc_silu(v.z); v.w = rc_silu(v.w); }
-                if (e < CH * RW) *reinterpret_cast<float4*>(da_sm + buf * CH * RW + e) = v;
-            }
-        } else {
-#pragma unroll
-            for (int k = 0; k < PER; k++) {
-                const int e = threadIdx.x + k * 32 * DA_WARPS;
-                if (e < CH * RW) da_sm[buf * CH * RW + e] = activated ? stage[k] : rc_silu(stage[k]);
-            }
-        }
-    };
-    const int chunks = (len + CH - 1) / CH;
-    if (chunks > 0) { load(0); store(0); }
+    if (chunks > 0) arrive(0);
     __syncthreads();
     for (int ch = 0; ch < chunks; ch++) {
         if (ch + 1 < chunks) load(ch + 1);
@@ -471,58 +503,44 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
             for (int k = 0; k < TB * VC; k++) acc[k] = 0.f;
             auto token = [&](int tb) {
                 const float* row = base + (t0 + tb) * RW;
-                float q[JD], k[JD], v[VC], ak[KEY ? JD : 1];
-                float a = dec;
-                if constexpr (JD % 4 == 0) {
-#pragma unroll
-                    for (int j = 0; j < JD; j += 4) {
-                        const float4 a = *reinterpret_cast<const float4*>(row + lane * JD + j);
-                        const float4 b = *reinterpret_cast<const float4*>(row + DP + lane * JD + j);
-                        q[j] = a.x; q[j + 1] = a.y; q[j + 2] = a.z; q[j + 3] = a.w;
-                        k[j] = b.x; k[j + 1] = b.y; k[j + 2] = b.z; k[j + 3] = b.w;
-                        if constexpr (KEY) {
-                            const float4 c = *reinterpret_cast<const float4*>(row + 2 * DP + lane * JD + j);
-                            ak[j] = c.x; ak[j + 1] = c.y; ak[j + 2] = c.z; ak[j + 3] = c.w;
-                        }
-                    }
-                } else if constexpr (JD == 2) {
-                    const float2 a = *reinterpret_cast<const float2*>(row + lane * 2);
-                    const float2 b = *reinterpret_cast<const float2*>(row + DP + lane * 2);
-                    q[0] = a.x; q[1] = a.y; k[0] = b.x; k[1] = b.y;
-                    if constexpr (KEY) {
-                        const float2 c = *reinterpret_cast<const float2*>(row + 2 * DP + lane * 2);
-                        ak[0] = c.x; ak[1] = c.y;
-                    }
-                } else {
-#pragma unroll
-                    for (int j = 0; j < JD; j++) {
-                        q[j] = row[lane * JD + j]; k[j] = row[DP + lane * JD + j];
-                        if constexpr (KEY) ak[j] = row[2 * DP + lane * JD + j];
-                    }
-                }
+                F2 q[NP], k[NP], ak[KEY ? NP : 1], v[NC];
+                rc_lane_values<JD>(row, lane, q);
+                rc_lane_values<JD>(row + DP, lane, k);
+                if constexpr (KEY) rc_lane_values<JD>(row + 2 * DP, lane, ak);
+                float2 ad = make_float2(dec, 1.f);
+                if constexpr (SSD) ad = *reinterpret_cast<const float2*>(da_coef + ((ch & 1) * CH + t0 + tb) * 2);
+                const F2 a = f2_pack(ad.x, ad.x);
+                float vf[VC];
                 if constexpr (VC % 4 == 0) {
 #pragma unroll
                     for (int c = 0; c < VC; c += 4) {
-                        const float4 a = *reinterpret_cast<const float4*>(row + VA + warp * VC + c);
-                        v[c] = a.x; v[c + 1] = a.y; v[c + 2] = a.z; v[c + 3] = a.w;
+                        const float4 x = *reinterpret_cast<const float4*>(row + VA + warp * VC + c);
+                        vf[c] = x.x; vf[c + 1] = x.y; vf[c + 2] = x.z; vf[c + 3] = x.w;
                     }
                 } else {
 #pragma unroll
-                    for (int c = 0; c < VC; c++) v[c] = row[VA + warp * VC + c];
+                    for (int c = 0; c < VC; c += 2) {
+                        const float2 x = *reinterpret_cast<const float2*>(row + VA + warp * VC + c);
+                        vf[c] = x.x; vf[c + 1] = x.y;
+                    }
                 }
                 if constexpr (SSD) {
-                    const float2 ad = *reinterpret_cast<const float2*>(da_coef + ((ch & 1) * CH + t0 + tb) * 2);
-                    a = ad.x;
 #pragma unroll
-                    for (int c = 0; c < VC; c++) v[c] *= ad.y;
+                    for (int c = 0; c < VC; c++) vf[c] *= ad.y;
                 }
 #pragma unroll
-                for (int j = 0; j < JD; j++) {
+                for (int c = 0; c < NC; c++) v[c] = JD == 1 ? f2_pack(vf[2 * c], vf[2 * c + 1]) : f2_pack(vf[c], vf[c]);
 #pragma unroll
-                    for (int c = 0; c < VC; c++) {
-                        s[c][j] = fmaf(KEY ? ak[KEY ? j : 0] : a, s[c][j], k[j] * v[c]);
-                        acc[tb * VC + c] = fmaf(s[c][j], q[j], acc[tb * VC + c]);
+                for (int c = 0; c < NC; c++) {
+                    F2 y;
+#pragma unroll
+                    for (int j = 0; j < NP; j++) {
+                        s[c][j] = f2_fma(KEY ? ak[KEY ? j : 0] : a, s[c][j], f2_mul(k[j], v[c]));
+                        y = j == 0 ? f2_mul(s[c][j], q[j]) : f2_fma(s[c][j], q[j], y);
                     }
+                    const float2 sum = f2_unpack(y);
+                    if constexpr (JD == 1) { acc[tb * VC + 2 * c] = sum.x; acc[tb * VC + 2 * c + 1] = sum.y; }
+                    else acc[tb * VC + c] = sum.x + sum.y;
                 }
             };
             // (a whole batch of tokens without a branch between them: their reads of shared memory are then in flight together)
@@ -546,8 +564,7 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
             }
             // the sum this lane holds: bit 16 of the lane chose the upper 16 of 32, bit 8 the upper 8 of those, ...: the lane's number
             // read from its highest bit down is the sum's index
-            const int mine = ((lane & 16) ? 16 : 0) + ((lane & 8) ? 8 : 0) + ((lane & 4) ? 4 : 0) + ((lane & 2) ? 2 : 0) + (lane & 1);
-            const int tb = mine / VC, c = mine % VC;
+            const int tb = lane / VC, c = lane % VC;
             if (t0 + tb < here && v0 + c < V) {
                 float y = acc[0];
                 if constexpr (SSD) y = fmaf(skip, base[(t0 + tb) * RW + VA + warp * VC + c], y);
@@ -555,28 +572,37 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
                 o[(size_t)(start + ch * CH + t0 + tb) * H * V + (size_t)h * V + v0 + c] = y;
             }
         }
-        if (ch + 1 < chunks) store((ch + 1) & 1);
+        if (ch + 1 < chunks) arrive(ch + 1);
         __syncthreads();
     }
-    if (whole) {
+    if constexpr (JD == 1) {
 #pragma unroll
-        for (int c = 0; c < VC; c++) {
-            if (lane * JD >= D || v0 + c >= V) continue;
-            float* p = st + at(lane * JD, c);
-            if constexpr (JD % 4 == 0) {
-#pragma unroll
-                for (int j = 0; j < JD; j += 4) *reinterpret_cast<float4*>(p + j) = make_float4(s[c][j], s[c][j + 1], s[c][j + 2], s[c][j + 3]);
-            } else if constexpr (JD == 2) {
-                *reinterpret_cast<float2*>(p) = make_float2(s[c][0], s[c][1]);
-            }
+        for (int c = 0; c < NC; c++) {
+            const float2 x = f2_unpack(s[c][0]);
+            if (lane < D && v0 + 2 * c < V) st[at(lane, 2 * c)] = x.x;
+            if (lane < D && v0 + 2 * c + 1 < V) st[at(lane, 2 * c + 1)] = x.y;
         }
     } else {
 #pragma unroll
-        for (int j = 0; j < JD; j++) {
-            const int d = lane * JD + j;
+        for (int c = 0; c < VC; c++) {
+            if (v0 + c >= V) continue;
+            float* p = st + at(lane * JD, c);
 #pragma unroll
-            for (int c = 0; c < VC; c++)
-                if (d < D && v0 + c < V) st[at(d, c)] = s[c][j];
+            for (int j = 0; j < JD; j += 2) {
+                const int d = lane * JD + j;
+                const float2 x = f2_unpack(s[c][j / 2]);
+                if (whole && JD % 4 == 0) {
+                    if (j % 4 == 0 && d < D) {
+                        const float2 y = f2_unpack(s[c][j / 2 + 1 < NP ? j / 2 + 1 : 0]);
+                        *reinterpret_cast<float4*>(p + j) = make_float4(x.x, x.y, y.x, y.y);
+                    }
+                } else if (whole) {
+                    if (d < D) *reinterpret_cast<float2*>(p + j) = x;
+                } else {
+                    if (d < D) p[j] = x.x;
+                    if (d + 1 < D) p[j + 1] = x.y;
+                }
+            }
         }
     }
     if constexpr (SSD)
@@ -626,7 +652,7 @@ static int launch_decay_scan(const float* proj, long long ldp, int q_col, int k_
 
 // proj [n][ldp] float32: q at q_col [H][D], k at k_col [H][D], v at v_col [H][V]; with `silu` their pre-activations (columns from the
 // first of q to the last of v, which a step of many tokens activates in place), else as they are; decay [H] float32; state
-// [slots][state_stride] float32, S [H][D][V];  o [n][H V] float32 receives the read-outs, times read_scale.
+// [slots][state_stride] float32, S [H][V][D];  o [n][H V] float32 receives the read-outs, times read_scale.
 XR_EXPORT int xr_decay_attention(float* proj, long long ldp, int q_col, int k_col, int v_col, const float* decay, float* state,
                                  long long state_stride, const int* seg_start, const int* seg_len, const int* seg_slot, float* o, int n, int n_seg,
                                  int H, int D, int V, int silu, float read_scale, cudaStream_t stream) {
