@@ -611,6 +611,10 @@ k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col
                                   blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
 }
 
+// Value columns a warp: two where the walk's length is what counts (few blocks, each with its SM to itself), four where there are more
+// blocks than the machine holds at once (half the reads of shared memory per state element).  A column's arithmetic is the same.
+static inline bool decay_scan_wide(int V, int H, int n_seg) { return (long long)((V + 15) / 16) * H * n_seg > 2LL * xr_sm_count(); }
+
 // bytes of shared memory a block of the walk takes: two chunks of CH tokens' rows
 static constexpr size_t decay_scan_smem(int JD, int VC, int CH, int KIND) {
     return (size_t)2 * CH * ((KIND == DS_KEY ? 3 : 2) * 32 * JD + VC * DA_WARPS) * sizeof(float);
@@ -640,9 +644,12 @@ static int launch_decay_scan(const float* proj, long long ldp, int q_col, int k_
         if (vec) DS1(JD, VC, CH, true);                                                                                                      \
         else DS1(JD, VC, CH, false);                                                                                                         \
     } while (0)
+    const bool wide = decay_scan_wide(V, H, n_seg);
     if (D <= 32) DS(1, 2, 16);
-    else if (D <= 64) DS(2, 2, 16);
-    else if (D <= 128) DS(4, 2, 16);
+    else if (D <= 64 && !wide) DS(2, 2, 16);
+    else if (D <= 64) DS(2, 4, 16);
+    else if (D <= 128 && !wide) DS(4, 2, 16);
+    else if (D <= 128) DS(4, 4, 16);
     else DS(8, 4, 8);
 #undef DS
 #undef DS1
@@ -814,9 +821,12 @@ XR_EXPORT int xr_ssd(const float* proj, long long ldp, int x_col, int dt_col, co
         if (vec) SS1(JD, VC, CK, true);                                                                                                      \
         else SS1(JD, VC, CK, false);                                                                                                         \
     } while (0)
+    const bool wide = decay_scan_wide(V, H, n_seg);
     if (N <= 32) SS(1, 2, 16);
-    else if (N <= 64) SS(2, 2, 16);
-    else if (N <= 128) SS(4, 2, 16);
+    else if (N <= 64 && !wide) SS(2, 2, 16);
+    else if (N <= 64) SS(2, 4, 16);
+    else if (N <= 128 && !wide) SS(4, 2, 16);
+    else if (N <= 128) SS(4, 4, 16);
     else SS(8, 4, 8);
 #undef SS
 #undef SS1
