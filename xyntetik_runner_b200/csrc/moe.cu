@@ -206,7 +206,8 @@ XR_EXPORT int xr_moe_plan(const int* ids, int* row_src, int* pair_row, int* tile
 
 // ---------------------------------------------------------------------------------------------
 // out[r] = h[row_src[r] / top] for the rows of tiles that hold any, zeros for rows of padding: the first product's
-// input in the order of the plan, for the tensor-core product (which reads its rows through a tensor map).
+// input in the order of the plan, for the tensor-core product (which reads its rows through a tensor map).  T: what a thread moves at a
+// time (an element, or 16 bytes of them; ldh and width are counted in it).
 // ---------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -219,7 +220,7 @@ k_moe_gather(const T* __restrict__ h, long long ldh, T* __restrict__ out, const 
     const int src = row_src[r];
     T* o = out + (size_t)r * width;
     if (src < 0) {
-        for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = xr_from_f32<T>(0.f);
+        for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = T{};
         return;
     }
     const T* a = h + (size_t)(src / top) * ldh;
@@ -229,9 +230,18 @@ k_moe_gather(const T* __restrict__ h, long long ldh, T* __restrict__ out, const 
 XR_EXPORT int xr_moe_gather(const void* h, int dtype, long long ldh, void* out, const int* row_src, const int* tile_group, int top,
                             int width, int align, int max_rows, cudaStream_t stream) {
     if (max_rows < 1 || width < 1 || top < 1 || align < 1) return XR_ERR_ARG;
-    if (dtype == XR_F32) xr_launch((k_moe_gather<float>), dim3(max_rows), dim3(256), 0, stream, (const float*)h, ldh, (float*)out, row_src, tile_group, top, width, align);
-    else if (dtype == XR_BF16) xr_launch((k_moe_gather<__nv_bfloat16>), dim3(max_rows), dim3(256), 0, stream, (const __nv_bfloat16*)h, ldh, (__nv_bfloat16*)out, row_src, tile_group, top, width, align);
-    else return XR_ERR_ARG;
+    if (dtype != XR_F32 && dtype != XR_BF16) return XR_ERR_ARG;
+    const int size = dtype == XR_F32 ? 4 : 2, per = 16 / size;
+#define GATHER(T, DIV)                                                                                                                       \
+    do {                                                                                                                                     \
+        const int units = width / (DIV), threads = units >= 256 ? 256 : (units + 31) / 32 * 32;                                              \
+        xr_launch((k_moe_gather<T>), dim3(max_rows), dim3(threads), 0, stream, (const T*)h, ldh / (DIV), (T*)out, row_src, tile_group, top,  \
+                  units, align);                                                                                                             \
+    } while (0)
+    if (width % per == 0 && ldh % per == 0 && !(((uintptr_t)h | (uintptr_t)out) & 15)) GATHER(uint4, per);
+    else if (dtype == XR_F32) GATHER(float, 1);
+    else GATHER(__nv_bfloat16, 1);
+#undef GATHER
     return xr_launch_status();
 }
 

@@ -371,8 +371,9 @@ __device__ __forceinline__ void rc_lane_values(const float* row, int lane, F2* o
     }
 }
 
+// (blocks an SM: one where the walk's length counts, whose loads then have the registers to run ahead; two where there are many blocks)
 template <int JD, int VC, int CH, bool VEC, int KIND>
-__global__ void __launch_bounds__(32 * DA_WARPS)
+__global__ void __launch_bounds__(32 * DA_WARPS, JD == 1 || (JD <= 4 && VC == 4) ? 2 : 1)
 k_decay_scan(const float* __restrict__ proj, long long ldp, int q_col, int k_col, int v_col, const float* __restrict__ decay,
              float* __restrict__ state, long long state_stride, const int* __restrict__ seg_start, const int* __restrict__ seg_len,
              const int* __restrict__ seg_slot, float* __restrict__ o, int H, int D, int V, int activated, SsdArgs ssd, KeyDecayArgs key) {
