@@ -222,7 +222,7 @@ FAMILIES = {
     "moe_gather": "grouped products (experts, per-head)", "heads_gather": "grouped products (experts, per-head)",
     "heads_scatter_gate": "grouped products (experts, per-head)",
     "mlstm": "mlstm recurrence", "route_topk": "routing", "moe_plan": "routing", "moe_gemm": "experts' products", "moe_combine": "experts' sum",
-    "delta": "delta recurrence", "head_norm_gate": "delta recurrence", "qk_norm_rope_store": "rotation + cache store",
+    "delta": "delta recurrence", "head_norm_gate": "gated norm of the recurrence", "qk_norm_rope_store": "rotation + cache store",
     "rmsnorm_act": "norms", "ssd": "state-space recurrence", "silu_gate_norm": "gated norm of the recurrence", "route_groups": "routing",
     "sigmoid_gate": "output gates", "stream_step": "stream kernels",
     "rglru": "gated linear recurrence", "decay_attention": "decay attention recurrence", "key_decay_attention": "key-decay attention recurrence", "norm_add": "norms", "depth_average": "stream kernels",
@@ -512,7 +512,7 @@ def _lilalorn_work(cfg, tokens, keys_per_token, decode):
     by_p += 2.0 * cfg.vocab * W
     by_n += tokens * W * (4 + 2)
     return {"attention": (fl_a, by_a), "products (tcgen05)": (fl_p, by_p), "norms": (0.0, by_n), "rotation + cache store": (0.0, by_r),
-            "decay attention recurrence": (fl_d, by_d), "key-decay attention recurrence": (fl_k, by_k), "delta recurrence": (0.0, by_h),
+            "decay attention recurrence": (fl_d, by_d), "key-decay attention recurrence": (fl_k, by_k), "gated norm of the recurrence": (0.0, by_h),
             "grouped products (experts, per-head)": (fl_e, by_e), "experts' sum": (0.0, by_c)}
 
 
